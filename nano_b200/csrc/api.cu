@@ -42,6 +42,7 @@ const DirFamily kDirFamilies[] = {
     {"Rakarax", nb_family_layered_create, "layered.cu"},
     {"Gokinex", nb_family_layered_create, "layered.cu"},
     {"Vumunex", nb_family_layered_create, "layered.cu"},
+    {"Kadesun", nb_family_layered_create, "layered.cu"},
 };
 }  // namespace
 

@@ -20,6 +20,11 @@
 // beside it, rotary positions on interleaved pairs, causal, ordinary softmax, output gate); feed-forward "dense" (exact gelu) or "moe"
 // (clamped gated experts chosen by their softmax scores, weighted on the way out, plus a shared expert); "loop" as below, without
 // the embedding added again.
+// "Kadesun" -- sequential sublayers that read the residual itself and are normed on the way out only, x <- x + rms_norm(sublayer(x)) w;
+// mixers "delta" (gated delta rule: fp32 matrix state per head, short convolutions, one decay per head and token, silu output gate) and
+// "parallel" (a grouped-query attention with query/key norm over the whole projection, rotary positions on half pairs, soft-capped
+// scores, a sink and one sigmoid gate per head, side by side with a gated delta rule whose decay is one number per key channel and whose
+// decay and output gate are low-rank products; each branch normed, then averaged); feed-forward "dense" (gated silu), or none.
 // "Famudra" -- parallel layers  x <- x + (mixer(shift(norm1 x)) + ff(norm2 x))  with scalar-gain RMS norms and a
 // token shift on the mixer input; mixers "rglru" (gelu branch x conv + real-gated linear recurrent unit) and "latent_attention"
 // (queries and keys/values through normed low-rank latents, no positions, causal softmax); feed-forward "moe" (top-k routed
@@ -54,6 +59,7 @@
 #include "layered_mixers.cuh"
 #include "layered_mixers2.cuh"
 #include "layered_mixers3.cuh"
+#include "layered_mixers4.cuh"
 #include "modeldir.h"
 #include "sample_host.h"
 
@@ -66,11 +72,12 @@ namespace {
 
 struct Weight { void *p = nullptr; uint32_t rows = 0, cols = 0; };
 
-enum MixerType { MIX_RGLRU = 0, MIX_LATENT_ATTN = 1, MIX_RETENTION = 2, MIX_WINDOW_SSM = 3, MIX_DIFF_ATTN = 4, MIX_SSD = 5 };
+enum MixerType { MIX_RGLRU = 0, MIX_LATENT_ATTN = 1, MIX_RETENTION = 2, MIX_WINDOW_SSM = 3, MIX_DIFF_ATTN = 4, MIX_SSD = 5, MIX_DELTA = 6, MIX_ATTN_DELTA = 7 };
 // how a layer combines its sublayers: Famudra's parallel form with a token shift and scalar-gain norms, or sequential sublayers
 // between an input norm and an output norm each (vector gains stored around zero)
 // or pre-norm sublayers over hyper-connected residual streams (bias-free layer norms)
-enum LayerForm { FORM_PARALLEL_SHIFT = 0, FORM_SANDWICH = 1, FORM_HYPER = 2 };
+// or sequential sublayers that read the residual itself and pass a norm on the way out (plain vector gains)
+enum LayerForm { FORM_PARALLEL_SHIFT = 0, FORM_SANDWICH = 1, FORM_HYPER = 2, FORM_POST = 3 };
 enum FfKind { FF_NONE = 0, FF_MOE = 1, FF_DENSE_POLY = 2, FF_DENSE_GLU = 3, FF_MOE_SCORED = 4, FF_DENSE_GELU = 5 };
 // the norms of the sequential form: unit RMS times a vector gain stored around zero, or Dynamic Tanh
 enum NormKind { NORM_RMS_ZERO = 0, NORM_DYT = 1 };
@@ -113,6 +120,15 @@ struct Layer {
     // state-space duality: proj = [z | x | B | C | dt]; H heads of vdim, mN states, G groups, m_taps, m_conv, m_conv_b, dt_b, A = exp(A_log)
     // per head, Dv per head; the output is normed in `parts` equal parts with the gain gn
     uint32_t parts = 0; float *gn = nullptr;
+    // output-normed form: gains after the mixer and after the feed-forward
+    float *pn1 = nullptr, *pn2 = nullptr;
+    // gated delta rule (MIX_DELTA, and one branch of MIX_ATTN_DELTA): dH heads of value size dVD over dG query/key heads of dD; columns of the
+    // joint product: convolved channels [q | k | v] from c_conv, step size c_b, decay c_a (a1 of rank ra, or one number per head), gate c_g
+    // (g1 of rank rg, or H VD numbers).  MIX_ATTN_DELTA: attention [q | k | v] from column 0, its gate at c_hg; out1 / out2: the gains of
+    // the branches' norms; mix_w: the weight of their sum
+    uint32_t dH = 0, dG = 0, dD = 0, dVD = 0, d_taps = 0, ra = 0, rg = 0, c_conv = 0, c_b = 0, c_a = 0, c_g = 0, c_hg = 0, a_half = 0;
+    float *d_conv = nullptr, *d_bias = nullptr, *d_rate = nullptr, *d_gain = nullptr, *qn = nullptr, *kn = nullptr, *out1 = nullptr, *out2 = nullptr, mix_w = 1.0f;
+    Weight a2, g2, d_o;
     // feed-forward
     int ff_kind = FF_NONE; float *act = nullptr;
     bool has_mlp = false, has_shared = false;
@@ -166,6 +182,9 @@ struct LayeredEngine : nb::EngineBase {
     // short portions of a Dynamic-Tanh design: the residual update that follows a sublayer rides on the sublayer's last product
     struct ResEpi { bool on = false; Dyt post{}, pre{}; float *out = nullptr, *keep = nullptr; } res;
     float *b_dpart = nullptr, *b_sseg = nullptr, *b_sdx = nullptr, *b_sdy = nullptr, *b_f2 = nullptr, *b_hg = nullptr, *b_sh2 = nullptr, *b_sg = nullptr, *b_wrow = nullptr; uint32_t *b_dtick = nullptr;
+    // gated delta rule: convolved channels of a short portion; what the preparation hands the scan; low-rank products; outputs before and after the gate
+    float *b_gcv = nullptr, *b_gq = nullptr, *b_gk = nullptr, *b_gv = nullptr, *b_gg = nullptr, *b_gsc = nullptr, *b_gsp = nullptr, *b_gt = nullptr, *b_go = nullptr, *b_ga = nullptr;
+    float *b_gpart = nullptr; uint32_t *b_gtick = nullptr;      // grouped-query attention: partials and tickets of the key splits
     uint32_t *ids_dev = nullptr, *want_dev = nullptr, *next_dev = nullptr, *tok_host = nullptr; uint8_t *seen = nullptr;
     uint32_t last_T = 0;
     uint32_t S = 1; float res_mult = 1.0f; float *xs = nullptr;      // hyper-connected form: streams, the model's residual multiplier, the streams [S][chunk][E]
@@ -549,10 +568,10 @@ int load_ssd(Loader &ld, const nb::Json *m, const std::string &p, Layer *L, uint
     return ld.put_f32(al, &L->A);
 }
 
-// gated feed-forward down(act(gate h) x (up h)): up = [gate | up] stacked
-int load_glu_dense(Loader &ld, const nb::Json *f, const std::string &p, Layer *L, uint32_t E) {
+// gated feed-forward down(act(gate h) x (up h)): up = [gate | up] stacked; act as in GemmArgs::glu (1: gelu_tanh, 2: silu)
+int load_glu_dense(Loader &ld, const nb::Json *f, const std::string &p, Layer *L, uint32_t E, uint32_t act) {
     if (!u32_of(f, "ff", &L->ff) || !L->ff) return fail(NB200_EINVAL, "%s: a dense feed-forward needs ff", p.c_str());
-    L->has_mlp = true; L->ff_kind = FF_DENSE_GLU;
+    L->has_mlp = true; L->ff_kind = FF_DENSE_GLU; L->glu_kind = act;
     int r;
     if ((r = ld.stacked({p + "gate", p + "up"}, {L->ff, L->ff}, E, &L->up))) return r;
     return ld.stacked({p + "down"}, {E}, L->ff, &L->down);
@@ -635,6 +654,104 @@ int load_dense_gelu(Loader &ld, const nb::Json *f, const std::string &p, Layer *
     int r;
     if ((r = ld.stacked({p + "up"}, {L->ff}, E, &L->up))) return r;
     return ld.stacked({p + "down"}, {E}, L->ff, &L->down);
+}
+
+// ---- gated delta rule, alone or beside a grouped-query attention: the rows of one joint product, collected in column order ----
+struct JointRows {
+    std::vector<float> all; uint32_t cols = 0;
+    int add(Loader &ld, const std::string &name, uint64_t rows, uint64_t E, uint32_t *at) {
+        if (at) *at = cols;
+        cols += (uint32_t)rows;
+        return append_rows(ld, name, rows, E, 0, rows, &all);
+    }
+    int put(Loader &ld, uint32_t E, Weight *w) {      // rows of zeros up to a multiple of 4: product rows start on 16-byte boundaries
+        cols = (cols + 3u) & ~3u;
+        all.resize((size_t)cols * E, 0.0f);
+        return ld.put_w(all, cols, E, w);
+    }
+};
+int rank_of(Loader &ld, const std::string &name, uint32_t *r) {
+    const nb::StTensor &t = ld.dir->tensors.find(name)->second;
+    if (t.shape.size() != 2 || !t.shape[0] || t.shape[0] > (1u << 20)) return fail(NB200_EINVAL, "tensor \"%s\" must be a matrix [rank, width]", name.c_str());
+    *r = (uint32_t)t.shape[0];
+    return 0;
+}
+// everything but the per-head columns of the joint product: sizes, [q | k | v] with their taps, decay, gate, output product
+int load_delta_rule(Loader &ld, const nb::Json *m, const std::string &p, Layer *L, uint32_t E, JointRows *J) {
+    if (!u32_of(m, "heads", &L->dH) || !u32_of(m, "kv_heads", &L->dG) || !u32_of(m, "dim", &L->dD) || !u32_of(m, "vdim", &L->dVD) || !u32_of(m, "conv", &L->d_taps))
+        return fail(NB200_EINVAL, "%s: a gated delta rule needs heads, kv_heads, dim, vdim and conv", p.c_str());
+    if (!L->dH || !L->dG || L->dH % L->dG || !L->dD || !L->dVD || !L->d_taps)
+        return fail(NB200_EINVAL, "%s: heads %u / kv_heads %u / dim %u / vdim %u / conv %u unusable", p.c_str(), L->dH, L->dG, L->dD, L->dVD, L->d_taps);
+    if (L->dD > kDeltaDim || L->dVD > 1024) return fail(NB200_EINVAL, "%s: dim %u above %u or vdim %u above 1024 has no delta-rule kernel", p.c_str(), L->dD, kDeltaDim, L->dVD);
+    const uint64_t H = L->dH, G = L->dG, D = L->dD, VD = L->dVD, K = L->d_taps;
+    int r;
+    if ((r = J->add(ld, p + "q", G * D, E, &L->c_conv)) || (r = J->add(ld, p + "k", G * D, E, nullptr)) || (r = J->add(ld, p + "v", H * VD, E, nullptr))) return r;
+    {   // taps of q, k and v, one channel range
+        std::vector<float> taps;
+        if ((r = append_rows(ld, p + "q.conv", G * D, K, 0, G * D, &taps)) || (r = append_rows(ld, p + "k.conv", G * D, K, 0, G * D, &taps)) ||
+            (r = append_rows(ld, p + "v.conv", H * VD, K, 0, H * VD, &taps)) || (r = ld.put_f32(taps, &L->d_conv))) return r;
+    }
+    // a tensor that is there says which form a part has: a1, a2: low-rank decay per key channel, else one per head; g1, g2: low-rank
+    // sigmoid gate, else a full silu gate
+    if (ld.dir->tensors.count(p + "a1")) {
+        if ((r = rank_of(ld, p + "a1", &L->ra)) || (r = J->add(ld, p + "a1", L->ra, E, &L->c_a)) || (r = ld.stacked({p + "a2"}, {H * D}, L->ra, &L->a2)) || (r = ld.vec(p + "dt_bias", {H * D}, &L->d_bias))) return r;
+    } else if ((r = ld.vec(p + "dt_bias", {H}, &L->d_bias))) return r;
+    if (ld.dir->tensors.count(p + "g1")) {
+        if ((r = rank_of(ld, p + "g1", &L->rg)) || (r = J->add(ld, p + "g1", L->rg, E, &L->c_g)) || (r = ld.stacked({p + "g2"}, {H * VD}, L->rg, &L->g2))) return r;
+    } else if ((r = J->add(ld, p + "g", H * VD, E, &L->c_g))) return r;
+    std::vector<float> al; std::vector<uint64_t> sh;
+    if ((r = ld.host_f32(p + "A_log", &al, &sh)) || (r = ld.expect(p + "A_log", sh, {H}))) return r;
+    for (float &v : al) v = (float)exp((double)v);          // the decay rate of a head: g = exp(-rate softplus(.))
+    if ((r = ld.put_f32(al, &L->d_rate)) || (r = ld.vec(p + "norm", {VD}, &L->d_gain))) return r;
+    return ld.stacked({p + "o"}, {E}, H * VD, &L->d_o);
+}
+// the columns that are one number per head come last
+int load_delta_heads(Loader &ld, const std::string &p, Layer *L, uint32_t E, JointRows *J) {
+    int r;
+    if (!L->ra && (r = J->add(ld, p + "a", L->dH, E, &L->c_a))) return r;
+    return J->add(ld, p + "b", L->dH, E, &L->c_b);
+}
+int load_delta(Loader &ld, const nb::Json *m, const std::string &p, Layer *L, uint32_t E) {
+    JointRows J; int r;
+    if ((r = load_delta_rule(ld, m, p, L, E, &J)) || (r = load_delta_heads(ld, p, L, E, &J))) return r;
+    return J.put(ld, E, &L->proj);
+}
+
+constexpr size_t kGqaSmemMax = 227 * 1024;
+inline int gqa_vj(uint32_t vdim) { return vdim <= 64 ? 1 : vdim <= 128 ? 2 : 4; }
+// grouped-query attention ("left") and gated delta rule ("right") on the same input.  Of the attention, by presence: rot, softcap, the
+// tensors q.norm / k.norm (gains of a norm over the whole projection), sink and g (one gate per head)
+int load_attn_delta(Loader &ld, const nb::Json *m, const std::string &p, Layer *L, uint32_t E, uint32_t positions) {
+    const nb::Json *lf = m->get("left"), *rt = m->get("right");
+    if (!lf || lf->t != nb::Json::Obj || !rt || rt->t != nb::Json::Obj) return fail(NB200_EINVAL, "%s: a parallel mixer needs left and right", p.c_str());
+    double sc;
+    if (!u32_of(lf, "heads", &L->H) || !u32_of(lf, "kv_heads", &L->G) || !u32_of(lf, "dim", &L->dim) || !u32_of(lf, "vdim", &L->vdim) || !lf->number("scale", &sc))
+        return fail(NB200_EINVAL, "%sleft: an attention needs heads, kv_heads, dim, vdim and scale", p.c_str());
+    L->scale = (float)sc;
+    if (!L->H || !L->G || L->H % L->G || !L->dim || !L->vdim) return fail(NB200_EINVAL, "%sleft: heads %u / kv_heads %u / dim %u / vdim %u unusable", p.c_str(), L->H, L->G, L->dim, L->vdim);
+    if (L->dim > 256 || L->vdim > 256) return fail(NB200_EINVAL, "%sleft: dim %u or vdim %u above 256 has no attention kernel", p.c_str(), L->dim, L->vdim);
+    int r;
+    if (lf->present("softcap")) { double c; if (!lf->number("softcap", &c) || !(c >= 0.0)) return fail(NB200_EINVAL, "%sleft: softcap must be a number >= 0", p.c_str()); L->softcap = (float)c; }
+    if (lf->present("rot")) {
+        const nb::Json *rot = lf->get("rot");
+        if (!u32_of(rot, "dims", &L->rot_dims) || L->rot_dims > L->dim || (L->rot_dims & 1u)) return fail(NB200_EINVAL, "%sleft: rot needs an even dims <= dim", p.c_str());
+        if (L->rot_dims && (r = rope_table(ld, rot, p, L->rot_dims, positions, &L->rot_tab))) return r;
+        L->a_half = L->rot_dims / 2u;
+    }
+    const uint64_t H = L->H, G = L->G, D = L->dim, VD = L->vdim;
+    L->RL = (uint32_t)((G * D + G * VD + 3u) & ~(uint64_t)3u);
+    const std::string q = p + "left.";
+    JointRows J;
+    if ((r = J.add(ld, q + "q", H * D, E, nullptr)) || (r = J.add(ld, q + "k", G * D, E, nullptr)) || (r = J.add(ld, q + "v", G * VD, E, nullptr)) ||
+        (r = load_delta_rule(ld, rt, p + "right.", L, E, &J))) return r;
+    L->has_gate = ld.dir->tensors.count(q + "g") != 0;
+    if (L->has_gate && (r = J.add(ld, q + "g", H, E, &L->c_hg))) return r;
+    if ((r = load_delta_heads(ld, p + "right.", L, E, &J)) || (r = J.put(ld, E, &L->proj))) return r;
+    if (ld.dir->tensors.count(q + "q.norm") && (r = ld.vec(q + "q.norm", {H * D}, &L->qn))) return r;
+    if (ld.dir->tensors.count(q + "k.norm") && (r = ld.vec(q + "k.norm", {G * D}, &L->kn))) return r;
+    if (ld.dir->tensors.count(q + "sink") && (r = ld.vec(q + "sink", {H}, &L->sink))) return r;
+    L->mix_w = 0.5f;
+    return (r = ld.stacked({q + "o"}, {E}, H * VD, &L->o)) ? r : (r = ld.vec(p + "left.out", {E}, &L->out1)) ? r : ld.vec(p + "right.out", {E}, &L->out2);
 }
 
 // connection weights of one sublayer, packed [in S | out S | mix S x S (from, to)]; without the tensors a single stream is the plain residual
@@ -1085,8 +1202,106 @@ int mix_ssd(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) {
     return last_product(e, plain(e->b_a, inner, L.o, e->d, E, T), T);
 }
 
+// ---- gated delta rule ----
+// from the rows of the joint product (e->b_p; short portions: convolved into e->b_gcv by its epilogue) to dst [T][E]
+int delta_branch(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx, float *dst) {
+    const uint32_t T = cx.T, H = L.dH, G = L.dG, D = L.dD, VD = L.dVD, P = L.proj.rows, C = 2 * G * D + H * VD;
+    const float qscale = (float)(1.0 / sqrt((double)D));
+    int r;
+    if (T <= kGemvMaxM) {
+        DeltaStepArgs a{e->b_gcv, e->b_p, P, L.c_b, L.c_a, L.c_g, L.ra ? L.a2.p : nullptr, L.rg ? L.g2.p : nullptr, L.ra, L.rg, L.d_bias, L.d_rate, L.d_gain,
+                        cx.st + run.st_S, e->b_ga, T, H, G, D, VD, qscale, e->eps, e->f32 ? 0u : 1u};
+        const size_t smem = delta_step_smem(D, VD);
+        const uint32_t want = std::max(128u, (VD + 3u) / 4u * 32u);
+#define DELTA_STEP(DCH) (e->f32 ? launch<DeltaStepArgs>(e, k_delta_step<float, DCH>, dim3(H), dim3(std::min(delta_step_threads(DCH), want)), smem, a) \
+                                : launch<DeltaStepArgs>(e, k_delta_step<__nv_bfloat16, DCH>, dim3(H), dim3(std::min(delta_step_threads(DCH), want)), smem, a))
+        if (D <= 32) r = DELTA_STEP(1);
+        else if (D <= 64) r = DELTA_STEP(2);
+        else if (D <= 128) r = DELTA_STEP(4);
+        else r = DELTA_STEP(8);
+#undef DELTA_STEP
+        return r ? r : gemm(e, plain(e->b_ga, H * VD, L.d_o, dst, e->E, T), 1, T);
+    }
+    if (L.ra && (r = gemm(e, plain(e->b_p + L.c_a, P, L.a2, e->b_gsp, H * D, T, L.d_bias, EPI_SOFTPLUS), 1, T))) return r;
+    if (L.rg && (r = gemm(e, plain(e->b_p + L.c_g, P, L.g2, e->b_gt, H * VD, T), 1, T))) return r;
+    const uint32_t chunks = (T + kDeltaChunk - 1u) / kDeltaChunk;
+    DeltaPrepArgs pa{e->b_p, P, L.c_conv, L.c_b, L.c_a, L.d_conv, cx.st + run.st_conv, L.d_taps, L.ra ? e->b_gsp : nullptr, L.d_bias, L.d_rate,
+                     e->b_gq, e->b_gk, e->b_gv, e->b_gg, e->b_gsc, T, H, G, D, VD, qscale};
+    if ((r = launch<DeltaPrepArgs>(e, k_delta_prep, dim3(chunks, H), dim3(32 * kDeltaChunk), 0, pa))) return r;
+    if (L.d_taps > 1) {
+        ConvArgs ca{e->b_p + L.c_conv, P, L.d_conv, nullptr, cx.st + run.st_conv, nullptr, T, C, L.d_taps, 0, 1};
+        if ((r = launch<ConvArgs>(e, k_conv_state, dim3((C + 127u) / 128u), dim3(128), 0, ca))) return r;
+    }
+    DeltaScanArgs sa{e->b_gq, e->b_gk, e->b_gv, e->b_gg, e->b_gsc, cx.st + run.st_S, e->b_go, T, H, G, D, VD, L.ra ? D : 1u};
+    const dim3 grid((VD + 15u) / 16u, H), block(128);
+    if (D <= 32) r = launch<DeltaScanArgs>(e, k_delta_scan<1>, grid, block, 0, sa);
+    else if (D <= 64) r = launch<DeltaScanArgs>(e, k_delta_scan<2>, grid, block, 0, sa);
+    else if (D <= 128) r = launch<DeltaScanArgs>(e, k_delta_scan<4>, grid, block, 0, sa);
+    else r = launch<DeltaScanArgs>(e, k_delta_scan<8>, grid, block, 0, sa);
+    if (r) return r;
+    RetOutArgs oa{e->b_go, L.rg ? e->b_gt : e->b_p + L.c_g, L.rg ? H * VD : P, e->b_ga, T, H, VD, e->eps, L.d_gain, L.rg ? 1u : 0u};
+    if ((r = launch<RetOutArgs>(e, k_retention_out, dim3((T * H + 7u) / 8u), dim3(256), 0, oa))) return r;
+    return gemm(e, plain(e->b_ga, H * VD, L.d_o, dst, e->E, T), 1, T);
+}
+// the joint product; for short portions the delta rule's convolution and silu are its epilogue
+int delta_joint(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) {
+    GemmArgs pj = plain(e->hm, e->E, L.proj, e->b_p, L.proj.rows, cx.T);
+    if (cx.T <= kGemvMaxM) {
+        pj.epi = EPI_CONV_RANGES;
+        pj.cr[0] = {L.c_conv, L.c_conv + 2 * L.dG * L.dD + L.dH * L.dVD, L.d_conv, nullptr, cx.st + run.st_conv, e->b_gcv, L.d_taps, 1};
+    }
+    return gemm(e, pj, 1, cx.T);
+}
+int mix_delta(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) {
+    int r;
+    return (r = delta_joint(e, L, run, cx)) ? r : delta_branch(e, L, run, cx, e->d);
+}
+
+// ---- grouped-query attention ----
+template <int VJ>
+int gqa_attn_launch(LayeredEngine *e, const GqaArgs &a) {
+    return launch<GqaArgs>(e, k_gqa_attn<VJ>, dim3((a.T * (a.H / a.G) + kGqaM - 1u) / kGqaM, a.G), dim3(256), gqa_attn_smem(a.D, VJ), a);
+}
+uint32_t gqa_hb(const Layer &L) { return std::min(L.H / L.G, kGqaHeads); }
+// from the rows of the joint product (q, k, v from column 0) to dst [T][E]
+int gqa_branch(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx, float *dst) {
+    const uint32_t T = cx.T, H = L.H, G = L.G, D = L.dim, VD = L.vdim, P = L.proj.rows;
+    GqaArgs a{e->b_p, P, 0u, H * D, H * D + G * D, L.c_hg, L.qn, L.kn, L.rot_tab, L.a_half, run.cache, cx.table, T, H, G, D, VD, L.RL, cx.pos0, cx.pos_ptr, e->eps,
+              L.scale, L.softcap, L.sink, L.has_gate ? 1u : 0u, e->b_a, 1u, e->b_gpart, e->b_gtick, gqa_hb(L)};
+    int r;
+    if (T <= kGemvMaxM) {      // a captured step does not know the position: blocks without a share of the keys leave at once
+        const uint32_t pages = ((cx.pos_ptr ? e->max_tokens : cx.pos0 + T) + kPage - 1u) / kPage;
+        a.nsplit = std::max(1u, std::min(kGqaSplitMax, pages));
+        const dim3 grid(a.nsplit, G * ((H / G + a.hb - 1u) / a.hb), T), block(256);
+        const size_t smem = gqa_decode_smem(D, VD);
+        const bool vec = ((D | VD | P) & 3u) == 0;
+        const uint32_t w = std::max(D, VD);
+#define GQA_DECODE(CH) (vec ? launch<GqaArgs>(e, k_gqa_decode<CH, true>, grid, block, smem, a) : launch<GqaArgs>(e, k_gqa_decode<CH, false>, grid, block, smem, a))
+        r = w <= 64 ? GQA_DECODE(2) : w <= 128 ? GQA_DECODE(4) : GQA_DECODE(8);
+#undef GQA_DECODE
+    } else {
+        if ((r = launch<GqaArgs>(e, k_qk_norm_rope, dim3(T), dim3(256), 0, a))) return r;
+        const int vj = gqa_vj(VD);
+        r = vj == 1 ? gqa_attn_launch<1>(e, a) : vj == 2 ? gqa_attn_launch<2>(e, a) : gqa_attn_launch<4>(e, a);
+    }
+    return r ? r : gemm(e, plain(e->b_a, H * VD, L.o, dst, e->E, T), 1, T);
+}
+// attention (e->d) and delta rule (e->d2, on a second stream) on the same input; the residual update norms and averages them
+int mix_attn_delta(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) {
+    int r;
+    if ((r = delta_joint(e, L, run, cx))) return r;
+    if (e->branch_streams) { CK(cudaEventRecord(e->ev_fork, e->stream)); e->cur = e->side; CK(cudaStreamWaitEvent(e->side, e->ev_fork, 0)); }
+    if ((r = delta_branch(e, L, run, cx, e->d2))) return r;
+    if (e->branch_streams) { CK(cudaEventRecord(e->ev_join, e->side)); e->cur = e->stream; }
+    if ((r = gqa_branch(e, L, run, cx, e->d))) return r;
+    if (e->branch_streams) CK(cudaStreamWaitEvent(e->stream, e->ev_join, 0));
+    return 0;
+}
+
 int mix(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) {
     switch (L.type) {
+        case MIX_DELTA: return mix_delta(e, L, run, cx);
+        case MIX_ATTN_DELTA: return mix_attn_delta(e, L, run, cx);
         case MIX_RGLRU: return mix_rglru(e, L, run, cx);
         case MIX_LATENT_ATTN: return mix_latent_attn(e, L, run, cx);
         case MIX_RETENTION: return mix_retention(e, L, run, cx);
@@ -1115,11 +1330,11 @@ int ff_glu_dense(LayeredEngine *e, const Layer &L, uint32_t T) {
     int r;
     if (T <= kGemvMaxM) {
         GemmArgs u = plain(e->h2, e->E, L.up, e->b_f2, L.ff, T);
-        u.N = L.ff; u.glu = 1u;
+        u.N = L.ff; u.glu = L.glu_kind;
         if ((r = gemm(e, u, 1, T))) return r;
     } else {
         if ((r = gemm(e, plain(e->h2, e->E, L.up, e->b_f, 2 * L.ff, T), 1, T))) return r;
-        GluArgs ga{e->b_f, 2 * L.ff, e->b_f2, L.ff, nullptr, T, L.ff, 0u};
+        GluArgs ga{e->b_f, 2 * L.ff, e->b_f2, L.ff, nullptr, T, L.ff, L.glu_kind == 2u ? 1u : 0u};
         if ((r = launch<GluArgs>(e, k_glu, dim3(ew_grid((size_t)T * L.ff)), dim3(256), 0, ga))) return r;
     }
     return last_product(e, plain(e->b_f2, L.ff, L.down, e->d, e->E, T), T);
@@ -1212,6 +1427,16 @@ int sandwich(LayeredEngine *e, const float *d, const float *w_post, const float 
     return launch<SandwichArgs>(e, k_sandwich, dim3(T), dim3(T <= kGemvMaxM && e->E >= 2048 ? 1024 : (T <= kGemvMaxM && e->E >= 1024 ? 512 : 256)), 0, a);
 }
 
+// x += rms_norm(e->d) w; for a two-branch mixer (two) what is normed is the weighted sum of its normed branches e->d and e->d2
+int post_norm(LayeredEngine *e, const Layer *two, const float *w, float *keep, uint32_t T) {
+    PostNormArgs a{e->x, e->d, two ? e->d2 : nullptr, two ? two->out1 : nullptr, two ? two->out2 : nullptr, w, two ? two->mix_w : 1.0f, keep, T, e->E, e->eps};
+    // a short portion is a few lone blocks: wide ones, so that a thread's chain of loads stays short
+    const uint32_t per = T <= kGemvMaxM ? 2u : 8u, threads = std::min(1024u, std::max(128u, (e->E / per + 31u) & ~31u));
+    if (e->E <= 2u * threads) return launch<PostNormArgs>(e, k_post_norm<2>, dim3(T), dim3(threads), 0, a);
+    if (e->E <= 8u * threads) return launch<PostNormArgs>(e, k_post_norm<8>, dim3(T), dim3(threads), 0, a);
+    return launch<PostNormArgs>(e, k_post_norm<0>, dim3(T), dim3(threads), 0, a);
+}
+
 // every layer run over T tokens (x already holds their embeddings) of the sequence in `slot`, whose first token sits at pos0
 // (+ *pos_ptr: a captured decode step keeps the position on the device and uses a fixed number of key splits)
 int run_layers(LayeredEngine *e, uint32_t slot, uint32_t T, uint32_t pos0, const uint32_t *pos_ptr = nullptr) {
@@ -1224,6 +1449,11 @@ int run_layers(LayeredEngine *e, uint32_t slot, uint32_t T, uint32_t pos0, const
         const Run &run = e->runs[ri];
         const Layer &L = e->layers[run.layer];
         float *keep = e->keep ? e->keep + ri * (size_t)e->chunk_cap * E : nullptr;
+        if (e->form == FORM_POST) {      // sublayers read x itself (e->hm and e->h2 are x)
+            if ((r = mix(e, L, run, cx)) || (r = post_norm(e, L.type == MIX_ATTN_DELTA ? &L : nullptr, L.pn1, L.has_mlp ? nullptr : keep, T))) return r;
+            if (L.has_mlp && ((r = ff_glu_dense(e, L, T)) || (r = post_norm(e, nullptr, L.pn2, keep, T)))) return r;
+            continue;
+        }
         if (e->form == FORM_HYPER) {
             // e->hm already holds the mixer's input (from the embedding step or the update before); every update also prepares the
             // input of the sublayer that follows (this layer's feed-forward, or the next run's mixer)
@@ -1352,7 +1582,7 @@ int head_rows(LayeredEngine *e, uint32_t nw, const uint32_t *want_dev = nullptr)
         e->launches++;
         return gemm(e, plain(e->b_xn, e->E, e->head, e->logits, e->V, nw), 1, nw);
     }
-    k_final_norm<<<nw, 256, 0, e->stream>>>(e->x, want_dev ? want_dev : e->want_dev, e->final_norm, e->b_xn, e->E, e->eps, e->form == FORM_SANDWICH ? 1u : 0u);
+    k_final_norm<<<nw, 256, 0, e->stream>>>(e->x, want_dev ? want_dev : e->want_dev, e->final_norm, e->b_xn, e->E, e->eps, e->form == FORM_SANDWICH ? 1u : e->form == FORM_POST ? 2u : 0u);
     CK(cudaGetLastError());
     e->launches++;
     return gemm(e, plain(e->b_xn, e->E, e->head, e->logits, e->V, nw), 1, nw);
@@ -1742,7 +1972,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
     int r;
     const nb::Json *arch = cfg.get("architecture");
     const std::string design = arch && arch->t == nb::Json::Str ? arch->str : "";
-    e->form = design == "Rakarax" || design == "Gokinex" ? FORM_SANDWICH : (design == "Vumunex" ? FORM_HYPER : FORM_PARALLEL_SHIFT);
+    e->form = design == "Rakarax" || design == "Gokinex" ? FORM_SANDWICH : design == "Vumunex" ? FORM_HYPER : design == "Kadesun" ? FORM_POST : FORM_PARALLEL_SHIFT;
     e->norm_kind = design == "Gokinex" ? NORM_DYT : NORM_RMS_ZERO;
     if ((r = ld.stacked({"embed"}, {e->V}, E, &e->embed)) || (r = ld.stacked({"head"}, {e->V}, E, &e->head))) return r;
     e->layers.resize(NL);
@@ -1777,7 +2007,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
             if (lj.present("mlp")) {
                 const nb::Json *f = lj.get("mlp"), *kind = f->get("kind");
                 if ((r = load_dyt(ld, p + "norm2", E, &L.d2)) || (r = load_dyt(ld, p + "norm2b", E, &L.d2b))) return r;
-                if (kind && kind->t == nb::Json::Str && kind->str == "dense") r = load_glu_dense(ld, f, p + "mlp.", &L, E);
+                if (kind && kind->t == nb::Json::Str && kind->str == "dense") r = load_glu_dense(ld, f, p + "mlp.", &L, E, 1u);
                 else if (kind && kind->t == nb::Json::Str && kind->str == "moe") r = load_moe_scored(ld, f, p + "mlp.", &L, E);
                 else return fail(NB200_EINVAL, "layer %u: feed-forward kind \"%s\" is not known", i, kind && kind->t == nb::Json::Str ? kind->str.c_str() : "?");
                 if (r) return r;
@@ -1812,6 +2042,27 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
                 else if (kind && kind->t == nb::Json::Str && kind->str == "moe") r = load_moe_scored(ld, f, p + "mlp.", &L, E, true);
                 else return fail(NB200_EINVAL, "layer %u: feed-forward kind \"%s\" is not known", i, kind && kind->t == nb::Json::Str ? kind->str.c_str() : "?");
                 if (r) return r;
+            }
+        }
+    } else if (e->form == FORM_POST) {
+        if ((r = ld.vec("final.norm", {E}, &e->final_norm))) return r;
+        const uint32_t page_tokens = ((max_tokens + kPage - 1) / kPage + std::max(1u, env_u32("NB200_MAX_SEQS", 8))) * kPage;      // every position the cache pages can hold
+        for (uint32_t i = 0; i < NL; i++) {
+            Run q; q.layer = i; e->runs.push_back(q);
+            const nb::Json &lj = layers->arr[i];
+            Layer &L = e->layers[i];
+            const std::string p = "l" + std::to_string(i) + ".";
+            const nb::Json *type = lj.get("type"), *mixer = lj.get("mixer");
+            if (!type || type->t != nb::Json::Str || !mixer || mixer->t != nb::Json::Obj) return fail(NB200_EINVAL, "layer %u needs \"type\" and \"mixer\"", i);
+            if ((r = ld.vec(p + "norm1", {E}, &L.pn1))) return r;
+            if (type->str == "delta") { L.type = MIX_DELTA; r = load_delta(ld, mixer, p + "mix.", &L, E); }
+            else if (type->str == "parallel") { L.type = MIX_ATTN_DELTA; r = load_attn_delta(ld, mixer, p + "mix.", &L, E, page_tokens); }
+            else return fail(NB200_EINVAL, "layer %u: mixer type \"%s\" is not known", i, type->str.c_str());
+            if (r) return r;
+            if (lj.present("mlp")) {
+                const nb::Json *f = lj.get("mlp"), *kind = f->get("kind");
+                if (!kind || kind->t != nb::Json::Str || kind->str != "dense") return fail(NB200_EINVAL, "layer %u: feed-forward kind \"%s\" is not known here", i, kind && kind->t == nb::Json::Str ? kind->str.c_str() : "?");
+                if ((r = ld.vec(p + "norm2", {E}, &L.pn2)) || (r = load_glu_dense(ld, f, p + "mlp.", &L, E, 2u))) return r;
             }
         }
     } else if (e->form == FORM_SANDWICH) {
@@ -1903,6 +2154,12 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
                 DM(q.cache, (size_t)e->n_pages * kPage * L.RS * 4);
                 CK(cudaMemset(q.cache, 0, (size_t)e->n_pages * kPage * L.RS * 4));
                 break;
+            case MIX_DELTA: case MIX_ATTN_DELTA:      // the convolution's tail over [q | k | v], the state [head][value column][key coordinate], key and value rows
+                q.st_conv = off; off += (size_t)(L.d_taps - 1) * (2 * L.dG * L.dD + L.dH * L.dVD);
+                off = (off + 3) & ~(size_t)3;
+                q.st_S = off; off += (size_t)L.dH * L.dVD * L.dD;
+                if (L.type == MIX_ATTN_DELTA) { DM(q.cache, (size_t)e->n_pages * kPage * L.RL * 4); CK(cudaMemset(q.cache, 0, (size_t)e->n_pages * kPage * L.RL * 4)); }
+                break;
             case MIX_RETENTION: q.st_S = off; off += (size_t)L.H * L.vdim * L.dim; break;
             default:          // window attention + selective scan: the tails of both convolutions, the scan state, a cache of key/value rows
                 q.st_conv = off; off += (size_t)(L.a_taps - 1) * (L.H + L.G) * L.dim;
@@ -1925,6 +2182,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
     uint32_t mC = 0, mZ = 0, mQR = 0, mQ = 0, mHR = 0, mOV = 0, mNE = 0, mTop = 0, mFF = 0, mSFF = 0;
     uint32_t sP = 0, sQK = 0, sXC = 0, sA = 0, sRO = 0, sDBC = 0, sF = 0;
     uint32_t sDP = 0, sDT = 0, sXC2 = 0, sY = 0, sF2 = 0; size_t sSS = 0, diff_smem[4] = {0, 0, 0, 0};      // differential attention, state-space duality, gated feed-forward
+    uint32_t dC = 0, dQ = 0, dV = 0, dGd = 0, dSc = 0, dSp = 0, dGt = 0, dPart = 0, dTick = 0; size_t gqa_smem[5] = {0, 0, 0, 0, 0};      // gated delta rule, grouped-query attention
     size_t win_smem[4] = {0, 0, 0, 0};      // most shared memory any layer asks of the window-attention instances, per value-column count
     for (const Run &q : e->runs) {
         const Layer &L = e->layers[q.layer];
@@ -1950,6 +2208,19 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
             sP = std::max(sP, inner + XW + L.H); sXC2 = std::max(sXC2, XW); sY = std::max(sY, inner); sA = std::max(sA, inner);
             sSS = std::max(sSS, (size_t)inner * L.mN);
         }
+        if (L.type == MIX_DELTA || L.type == MIX_ATTN_DELTA) {
+            sP = std::max(sP, L.proj.rows);
+            dC = std::max(dC, 2 * L.dG * L.dD + L.dH * L.dVD); dQ = std::max(dQ, L.dG * L.dD); dV = std::max(dV, L.dH * L.dVD);
+            dGd = std::max(dGd, L.ra ? L.dH * L.dD : L.dH); dSc = std::max(dSc, L.dH * kDeltaSc);
+            if (L.ra) dSp = std::max(dSp, L.dH * L.dD);
+            if (L.rg) dGt = std::max(dGt, L.dH * L.dVD);
+        }
+        if (L.type == MIX_ATTN_DELTA) {
+            sA = std::max(sA, L.H * L.vdim); dPart = std::max(dPart, L.H * (L.vdim + 2)); dTick = std::max(dTick, L.G * ((L.H / L.G + gqa_hb(L) - 1u) / gqa_hb(L)));
+            const int vj = gqa_vj(L.vdim);
+            if (gqa_attn_smem(L.dim, vj) > kGqaSmemMax) return fail(NB200_EINVAL, "attention with %u query/key and %u value coordinates does not fit the attention kernel's shared memory", L.dim, L.vdim);
+            gqa_smem[vj] = std::max(gqa_smem[vj], gqa_attn_smem(L.dim, vj));
+        }
         if (L.ff_kind == FF_DENSE_GLU) { sF = std::max(sF, 2 * L.ff); sF2 = std::max(sF2, L.ff); }
     }
     if (diff_smem[0] > 48 * 1024 && (r = diff_attn_optin_v<1>((int)diff_smem[0]))) return r;
@@ -1960,6 +2231,19 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
         DM(e->b_dpart, (size_t)kGemvMaxM * kSplitMax * sDP * 4);
         DM(e->b_dtick, (size_t)kGemvMaxM * sDT * 4);
         CK(cudaMemset(e->b_dtick, 0, (size_t)kGemvMaxM * sDT * 4));
+    }
+    if (dC) {
+        DM(e->b_gcv, (size_t)kGemvMaxM * dC * 4); DM(e->b_gq, T * dQ * 4); DM(e->b_gk, T * dQ * 4); DM(e->b_gv, T * dV * 4); DM(e->b_gg, T * dGd * 4);
+        DM(e->b_gsc, (T + kDeltaChunk - 1) / kDeltaChunk * dSc * 4); DM(e->b_go, T * dV * 4); DM(e->b_ga, T * dV * 4);
+        if (dSp) DM(e->b_gsp, T * dSp * 4);
+        if (dGt) DM(e->b_gt, T * dGt * 4);
+    }
+    if (dPart) {
+        DM(e->d2, T * E * 4); DM(e->b_gpart, (size_t)kGemvMaxM * kGqaSplitMax * dPart * 4); DM(e->b_gtick, (size_t)kGemvMaxM * dTick * 4);
+        CK(cudaMemset(e->b_gtick, 0, (size_t)kGemvMaxM * dTick * 4));
+        if (gqa_smem[1] > 48 * 1024) CK(cudaFuncSetAttribute((const void *)k_gqa_attn<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gqa_smem[1]));
+        if (gqa_smem[2] > 48 * 1024) CK(cudaFuncSetAttribute((const void *)k_gqa_attn<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gqa_smem[2]));
+        if (gqa_smem[4] > 48 * 1024) CK(cudaFuncSetAttribute((const void *)k_gqa_attn<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gqa_smem[4]));
     }
     if (sSS) DM(e->b_sseg, (size_t)kRetSegs * sSS * 4);
     if (sXC2) DM(e->b_sdx, T * sXC2 * 4);
@@ -2001,7 +2285,9 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
         if (L.ff_kind == FF_MOE_SCORED) { mFF2 = std::max(mFF2, 2 * L.top * L.ff); mSFF2 = std::max(mSFF2, 2 * L.sff); }
     }
     if (e->form == FORM_HYPER) DM(e->xs, (size_t)e->S * T * E * 4);
-    DM(e->x, T * E * 4); DM(e->hm, T * E * 4); DM(e->h2, T * E * 4); DM(e->d, T * E * 4);
+    DM(e->x, T * E * 4); DM(e->d, T * E * 4);
+    if (e->form == FORM_POST) { e->hm = e->x; e->h2 = e->x; }      // no input norms: a sublayer reads the residual
+    else { DM(e->hm, T * E * 4); DM(e->h2, T * E * 4); }
     if (e->keep_x0) DM(e->x0, T * E * 4);
     if (mC) { DM(e->b_yx, T * 2 * mC * 4); DM(e->b_u, T * mC * 4); DM(e->b_g, T * 2 * mC * 4); DM(e->b_sy, T * mC * 4); }
     if (mZ) {

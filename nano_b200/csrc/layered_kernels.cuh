@@ -22,7 +22,7 @@
 //                        k_combine (weighted sum in choice order + shared expert + mixer output -> residual)
 //
 // More mechanisms (position table, sandwich norms, rotary positions, retention, window attention, selective scan, PolyNorm) live in
-// layered_mixers.cuh under the same rules.
+// layered_mixers.cuh and layered_mixers2 / 3 / 4.cuh under the same rules.
 //
 // What is fp32 here regardless of the weight type: the residual stream, every norm, router logits, attention scores / weights /
 // accumulators, gates, decays and the recurrent state.  bf16 enters only as a matrix-product operand.
@@ -1179,7 +1179,7 @@ __global__ void k_combine(const CombineArgs a) {
 }
 
 // scalar-gain RMS norm of the rows whose logits are asked for: out[i] = x[want[i]] / rms * g
-// (vec: the gain is a vector stored around zero, out = x / rms * (1 + g[i]))
+// (vec 1: the gain is a vector stored around zero, out = x / rms * (1 + g[i]); vec 2: a plain vector, out = x / rms * g[i])
 __global__ void __launch_bounds__(256) k_final_norm(const float *__restrict__ x, const uint32_t *__restrict__ want, const float *__restrict__ g,
                                                     float *__restrict__ out, uint32_t E, float eps, uint32_t vec) {
     pdl_enter();
@@ -1190,7 +1190,7 @@ __global__ void __launch_bounds__(256) k_final_norm(const float *__restrict__ x,
     s = block_sum(s, red);
     const float rinv = 1.0f / sqrtf(s / (float)E + eps) * 1.0f;
     const float gv = vec ? 0.0f : *g;
-    for (uint32_t i = threadIdx.x; i < E; i += blockDim.x) out[(size_t)blockIdx.x * E + i] = xt[i] * rinv * (vec ? 1.0f + g[i] : gv);
+    for (uint32_t i = threadIdx.x; i < E; i += blockDim.x) out[(size_t)blockIdx.x * E + i] = xt[i] * rinv * (vec ? (vec == 2u ? g[i] : 1.0f + g[i]) : gv);
 }
 
 // greedy choice with the repetition penalty of the generation hosts: logits of ids seen before are divided (positive) or multiplied
