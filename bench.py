@@ -848,6 +848,91 @@ def vumunex_bench(args):
                       "clocks": clocks, "sizes": out}))
 
 
+# --------------------------------------------------------------------------------------------------
+# --design kadesun: the same two measurements for the Kadesun design (grouped-query attention beside a gated delta rule with per-channel
+# decays, gated delta rule alone, gated dense feed-forward, norms on the way out of a sublayer only) beside the closest model of the
+# same runtime, Rakarax (the other design with two-sided mixers: grouped-query window attention + selective scan; retention; dense
+# feed-forward), at equal width and depth.
+# --------------------------------------------------------------------------------------------------
+KADESUN_SIZES = {
+    # name: (width, layers, attention heads, kv heads, dim, vdim, delta heads beside the attention, delta heads alone, kv heads alone, dim, vdim, low ranks, ff)
+    "w1024": (1024, 8, 16, 4, 64, 64, 8, 8, 8, 128, 128, 64, 3072),
+    "w2048": (2048, 8, 16, 4, 128, 128, 16, 16, 8, 128, 128, 128, 6144),
+}
+
+
+def kadesun_model(name):
+    from nano_b200 import modeldir as md
+    E_, L, H, G, D, VD, RH, DH, DG, RD, RVD, rank, ff = KADESUN_SIZES[name]
+    par = {"left": {"heads": H, "kv_heads": G, "dim": D, "vdim": VD, "scale": D ** -0.5, "softcap": 50.0, "rot": {"dims": D, "base": 500000.0}},
+           "right": {"heads": RH, "kv_heads": RH, "dim": RD, "vdim": RVD, "conv": 4}}
+    layers = [("parallel", par, ff) if i % 2 == 0 else ("delta", {"heads": DH, "kv_heads": DG, "dim": RD, "vdim": RVD, "conv": 4}, ff) for i in range(L)]
+    cfg = md.kadesun_config(FAMUDRA_VOCAB, E_, layers)
+    cfg["_rank"] = rank          # not read by the engine: the low ranks are the tensors' shapes
+    path = os.path.join(os.environ.get("NB200_MODEL_CACHE", "/tmp/nb200_models"), f"kadesun-{name}")
+    if not os.path.exists(os.path.join(path, "model.safetensors")):
+        md.write_model_dir(path + ".part", cfg, md.kadesun_random(cfg, 0, decay_rank=rank, gate_rank=rank))
+        os.replace(path + ".part", path)
+    return path, cfg
+
+
+def kadesun_decode_bytes(cfg, pos, wbytes=2):
+    """Algorithmic HBM bytes of one decoded token at position pos: every matrix once, the fp32 states read and written, the fp32 key and
+    value rows of every earlier position, the head."""
+    E_ = cfg["width"]; R = cfg["_rank"]; b = 0.0
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        d = m if L["type"] == "delta" else m["right"]
+        H, G, D, VD = d["heads"], d["kv_heads"], d["dim"], d["vdim"]
+        b += wbytes * (2 * G * D + 2 * H * VD + H) * E_ + 8.0 * H * D * VD          # q, k, v, o, step size; the state
+        if L["type"] == "delta":
+            b += wbytes * (H * VD + H) * E_
+        else:
+            a = m["left"]
+            b += wbytes * (2 * R * E_ + R * H * (D + VD))
+            b += wbytes * (a["heads"] * (a["dim"] + a["vdim"] + 1) + a["kv_heads"] * (a["dim"] + a["vdim"])) * E_ + 4.0 * a["kv_heads"] * (a["dim"] + a["vdim"]) * (pos + 1)
+        if L.get("mlp"):
+            b += wbytes * 3 * E_ * L["mlp"]["ff"]
+    return b + wbytes * cfg["vocab"] * E_
+
+
+def kadesun_flops_per_token(cfg, ctx):
+    fl = 2.0 * (kadesun_decode_bytes(cfg, 0, 1) - cfg["vocab"] * cfg["width"])
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        d = m if L["type"] == "delta" else m["right"]
+        fl -= 16.0 * d["heads"] * d["dim"] * d["vdim"]          # the state's bytes are no products
+        fl += 7.0 * d["heads"] * d["dim"] * d["vdim"]           # decay, S^T k, k u^T, S^T q
+        if L["type"] == "parallel":
+            a = m["left"]
+            fl += 2.0 * a["heads"] * (a["dim"] + a["vdim"]) * ctx
+    return fl
+
+
+def kadesun_bench(args):
+    from nano_b200 import engine as E
+    hbm, hbm_src = peaks()
+    try:
+        tf = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    except Exception:
+        tf = 1590.0
+    ctx, n_dec, T = 1024, 128, 2048
+    sampler = ClockSampler(0); sampler.start()
+    out = {}
+    for name in (args.sizes.split(",") if args.sizes else sorted(KADESUN_SIZES)):
+        path, cfg = kadesun_model(name)
+        row = layered_modes(E, path, FAMUDRA_VOCAB, ctx, n_dec, T, args, hbm, tf, lambda pos, wb: kadesun_decode_bytes(cfg, pos, wb), lambda c: kadesun_flops_per_token(cfg, c))
+        ppath, pcfg = rakarax_model(name)          # the closest model: the same runtime's Rakarax at equal width and depth
+        args_bf16 = argparse.Namespace(**{**vars(args), "with_f32": False})
+        row["peer_rakarax"] = layered_modes(E, ppath, FAMUDRA_VOCAB, ctx, n_dec, T, args_bf16, hbm, tf, lambda pos, wb: rakarax_decode_bytes(pcfg, pos, wb), lambda c: rakarax_flops_per_token(pcfg, c))["bf16"]
+        out[name] = row
+    clocks = sampler.stop()
+    print(json.dumps({"design": "kadesun", "unit": "tokens/s", "n_gpus": 1, "data": "synthetic (random weights)", "peaks": {"hbm_gbs": hbm, "hbm_source": hbm_src, "bf16_tflops": tf},
+                      "config": {"decode": f"greedy device loop, {n_dec} tokens after a {ctx}-token prompt, batch 1", "prefill": f"one portion of {T} tokens into an empty sequence",
+                                 "timing": "CUDA events on the engine's stream after warm-up", "l2": "fractions are against HBM although the weights of one token fit the 126 MB L2 at w1024"},
+                      "clocks": clocks, "sizes": out}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -864,7 +949,7 @@ def main():
     ap.add_argument("--no-pdl", action="store_true")
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--no-stream", action="store_true", help="forbid the streaming kernel")
-    ap.add_argument("--design", default=None, choices=["famudra", "rakarax", "gokinex", "vumunex"], help="measure a model-folder design instead of the headline workload (its own JSON line)")
+    ap.add_argument("--design", default=None, choices=["famudra", "rakarax", "gokinex", "vumunex", "kadesun"], help="measure a model-folder design instead of the headline workload (its own JSON line)")
     ap.add_argument("--sizes", default=None, help="--design: comma-separated size names (default: all)")
     ap.add_argument("--with-f32", action="store_true", help="--design: also time the true-32-bit mode")
     args = ap.parse_args()
@@ -879,6 +964,9 @@ def main():
         return
     if args.design == "gokinex":
         gokinex_bench(args)
+        return
+    if args.design == "kadesun":
+        kadesun_bench(args)
         return
     args.warmup = max(args.warmup, 3) if args.impl == "b200" else args.warmup
 

@@ -1211,10 +1211,9 @@ int delta_branch(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx
     if (T <= kGemvMaxM) {
         DeltaStepArgs a{e->b_gcv, e->b_p, P, L.c_b, L.c_a, L.c_g, L.ra ? L.a2.p : nullptr, L.rg ? L.g2.p : nullptr, L.ra, L.rg, L.d_bias, L.d_rate, L.d_gain,
                         cx.st + run.st_S, e->b_ga, T, H, G, D, VD, qscale, e->eps, e->f32 ? 0u : 1u};
-        const size_t smem = delta_step_smem(D, VD);
         const uint32_t want = std::max(128u, (VD + 3u) / 4u * 32u);
-#define DELTA_STEP(DCH) (e->f32 ? launch<DeltaStepArgs>(e, k_delta_step<float, DCH>, dim3(H), dim3(std::min(delta_step_threads(DCH), want)), smem, a) \
-                                : launch<DeltaStepArgs>(e, k_delta_step<__nv_bfloat16, DCH>, dim3(H), dim3(std::min(delta_step_threads(DCH), want)), smem, a))
+#define DELTA_STEP(DCH) (e->f32 ? launch<DeltaStepArgs>(e, k_delta_step<float, DCH>, dim3(H), dim3(std::min(delta_step_threads(DCH), want)), delta_step_smem(DCH, VD), a) \
+                                : launch<DeltaStepArgs>(e, k_delta_step<__nv_bfloat16, DCH>, dim3(H), dim3(std::min(delta_step_threads(DCH), want)), delta_step_smem(DCH, VD), a))
         if (D <= 32) r = DELTA_STEP(1);
         else if (D <= 64) r = DELTA_STEP(2);
         else if (D <= 128) r = DELTA_STEP(4);

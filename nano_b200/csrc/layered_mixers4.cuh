@@ -747,7 +747,7 @@ struct DeltaStepArgs {
     const float *cv; const float *p; uint32_t ld, b0, a0, g0; const void *a2, *g2; uint32_t ra, rg; const float *dt_bias, *rate, *gain;
     float *S; float *out; uint32_t T, H, G, D, VD; float qscale, eps; uint32_t round_a;
 };
-inline size_t delta_step_smem(uint32_t D, uint32_t VD) { return ((size_t)3 * kGemvMaxM * ((D + 31u) & ~31u) + (size_t)2 * kGemvMaxM * VD) * 4; }
+inline size_t delta_step_smem(int dch, uint32_t VD) { return ((size_t)3 * kGemvMaxM * (uint32_t)dch * 32u + (size_t)2 * kGemvMaxM * VD) * 4; }      // dch: the instance's, DCH
 // dot products of one weight row with up to kGemvMaxM rows of x (stride ld), 8 lanes per row; every lane gets the totals.  vec: 16-byte
 // loads of both operands are aligned
 template <typename WT>

@@ -1,5 +1,5 @@
-"""Model folders (config.json + model.safetensors) from the Python side: a writer, and random-weight Famudra, Rakarax, Gokinex and Vumunex models for
-the benchmarks and tests.  The reader the engine uses is native (csrc/modeldir.cu); nothing here is on the compute path.
+"""Model folders (config.json + model.safetensors) from the Python side: a writer, and random-weight Famudra, Rakarax, Gokinex, Vumunex and
+Kadesun models for the benchmarks and tests.  The reader the engine uses is native (csrc/modeldir.cu); nothing here is on the compute path.
 
 A safetensors file is an 8-byte little-endian header length, that many bytes of JSON (name -> dtype, shape, data_offsets) and
 the tensor bytes.
@@ -316,4 +316,61 @@ def vumunex_random(config: dict, seed: int = 0, gain: float = 1.0, layer_scale: 
             if S is not None:
                 t[p + f"hc{q}.in"] = vecn(S, 0.2, 0.6); t[p + f"hc{q}.out"] = vecn(S, 0.5, 1.5)
                 t[p + f"hc{q}.mix"] = bf16_round((np.eye(S) * 0.9 + 0.1 * rng.standard_normal((S, S))).astype(np.float32))
+    return t
+
+
+def kadesun_config(vocab: int, width: int, layers, eps: float = 1e-5) -> dict:
+    """layers: list of (type, mixer, ff).
+    type "delta": mixer {heads, kv_heads, dim, vdim, conv}; type "parallel": mixer {left: {heads, kv_heads, dim, vdim, scale, softcap,
+    rot: {dims, base}}, right: {heads, kv_heads, dim, vdim, conv}}; ff: width of the dense feed-forward, or None for a layer without one."""
+    out = [{"type": kind, "mixer": json.loads(json.dumps(mixer)), "mlp": {"kind": "dense", "ff": ff} if ff else None} for kind, mixer, ff in layers]
+    return {"architecture": "Kadesun", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": out}
+
+
+def kadesun_random(config: dict, seed: int = 0, gain: float = 1.0, decay_rank: int = 12, gate_rank: int = 20) -> Dict[str, np.ndarray]:
+    """Random weights (bfloat16-representable fp32 arrays) for a Kadesun config: projections ~ N(0, gain^2 / fan_in); decay_rank,
+    gate_rank: inner sizes of the low-rank decay and output gate of the parallel mixers."""
+    rng = np.random.default_rng(seed)
+    E, V = config["width"], config["vocab"]
+
+    def lin(o, i, g=1.0):
+        return bf16_round((rng.standard_normal((o, i), dtype=np.float32) * (gain * g / np.sqrt(i))).astype(np.float32))
+
+    def vecn(n, lo, hi):
+        return bf16_round(rng.uniform(lo, hi, size=n).astype(np.float32))
+
+    t = {"embed": bf16_round(rng.standard_normal((V, E), dtype=np.float32)), "head": lin(V, E), "final.norm": vecn(E, 0.7, 1.3)}
+
+    def delta(p, m, low_rank):
+        H, G, D, VD, K = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+        for n, rows in (("q", G * D), ("k", G * D), ("v", H * VD)):
+            t[p + n] = lin(rows, E, 1.5); t[p + n + ".conv"] = vecn((rows, K), -0.7, 0.9)
+        t[p + "b"] = lin(H, E)
+        t[p + "A_log"] = bf16_round(np.log(rng.uniform(0.1, 4.0, size=H)).astype(np.float32))
+        t[p + "norm"] = vecn(VD, 0.6, 1.4); t[p + "o"] = lin(E, H * VD)
+        if low_rank:
+            t[p + "a1"] = lin(decay_rank, E); t[p + "a2"] = lin(H * D, decay_rank, 1.5); t[p + "dt_bias"] = vecn(H * D, -6.0, 0.0)
+            t[p + "g1"] = lin(gate_rank, E); t[p + "g2"] = lin(H * VD, gate_rank, 1.5)
+        else:
+            t[p + "a"] = lin(H, E); t[p + "dt_bias"] = vecn(H, -6.0, 0.0); t[p + "g"] = lin(H * VD, E, 1.5)
+
+    for i, L in enumerate(config["layers"]):
+        p = f"l{i}."
+        t[p + "norm1"] = vecn(E, 0.4, 0.9)
+        m = L["mixer"]
+        if L["type"] == "delta":
+            delta(p + "mix.", m, False)
+        else:
+            a = m["left"]
+            H, G, D, VD = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            q = p + "mix.left."
+            t[q + "q"] = lin(H * D, E); t[q + "k"] = lin(G * D, E); t[q + "v"] = lin(G * VD, E)
+            t[q + "q.norm"] = vecn(H * D, 0.7, 1.6); t[q + "k.norm"] = vecn(G * D, 0.7, 1.6)
+            t[q + "sink"] = vecn(H, -1.0, 2.0); t[q + "g"] = lin(H, E, 1.5); t[q + "o"] = lin(E, H * VD)
+            delta(p + "mix.right.", m["right"], True)
+            t[p + "mix.left.out"] = vecn(E, 0.6, 1.4); t[p + "mix.right.out"] = vecn(E, 0.6, 1.4)
+        f = L.get("mlp")
+        if f:
+            t[p + "norm2"] = vecn(E, 0.4, 0.9)
+            t[p + "mlp.gate"] = lin(f["ff"], E, 1.5); t[p + "mlp.up"] = lin(f["ff"], E); t[p + "mlp.down"] = lin(E, f["ff"])
     return t

@@ -161,3 +161,58 @@ def test_vumunex_oracle_is_causal_windowed_and_routed():
     g = np.array([[3.0, -3.0]])
     e = O.expert({"e.gate": np.eye(2), "e.up": np.eye(2), "e.down": np.eye(2)}, "e.", g, 1.0)
     assert np.allclose(e, [[1.0 * O.sigmoid(1.702) * 2.0, -3.0 * O.sigmoid(-3.0 * 1.702) * 0.0]])      # the gate is capped from above only, the other branch on both sides
+
+
+KAD_LEFT = {"heads": 4, "kv_heads": 2, "dim": 8, "vdim": 6, "scale": 0.4, "softcap": 5.0, "rot": {"dims": 4, "base": 100.0}}
+KAD_DELTA = {"heads": 4, "kv_heads": 2, "dim": 6, "vdim": 10, "conv": 3}
+
+
+@pytest.mark.skipif(E.device_count() > 0, reason="box has a GPU")
+def test_kadesun_folder_reaches_the_layered_family(tmp_path):
+    cfg = md.kadesun_config(16, 8, [("delta", KAD_DELTA, None), ("parallel", {"left": KAD_LEFT, "right": KAD_DELTA}, 12)])
+    w = md.kadesun_random(cfg, decay_rank=3, gate_rank=5)
+    assert w["l0.mix.dt_bias"].shape == (4,) and w["l1.mix.right.dt_bias"].shape == (24,) and w["l1.mix.right.g2"].shape == (40, 5) and "l0.norm2" not in w
+    p = md.write_model_dir(str(tmp_path / "k"), cfg, w)
+    with pytest.raises(E.NB200Error, match="no CUDA device"):
+        E.Engine(p, 16)
+
+
+def test_kadesun_oracle_is_causal_and_follows_the_delta_rule():
+    """The plain restatement itself: a prefix gives the same logits; the recurrence overwrites what a key held, its read-out sees the
+    present write, and a state carried over equals one pass; decays act on the key coordinates; the sink takes weight away; the
+    convolution's last tap is the present token's."""
+    import kadesun_oracle as O
+    rng = np.random.default_rng(0)
+    cfg = md.kadesun_config(20, 16, [("parallel", {"left": KAD_LEFT, "right": KAD_DELTA}, 12), ("delta", KAD_DELTA, None)])
+    w = md.kadesun_random(cfg, 3)
+    t = rng.integers(0, 20, 24)
+    full = O.forward(cfg, w, t)
+    assert np.allclose(O.forward(cfg, w, t[:10]), full[:10], atol=1e-12)
+    q, k, v = rng.standard_normal((6, 2, 5)), O.unit(rng.standard_normal((6, 2, 5))), rng.standard_normal((6, 2, 3))
+    beta, g = rng.uniform(0, 1, (6, 2)), rng.uniform(0.2, 1, (6, 2, 5))
+    o, S = O.delta_recurrence(q, k, v, beta, g)
+    assert np.allclose(o[0, 1], beta[0, 1] * (q[0, 1] @ k[0, 1]) * v[0, 1])
+    o1, S1 = O.delta_recurrence(q[:4], k[:4], v[:4], beta[:4], g[:4])
+    o2, S2 = O.delta_recurrence(q[4:], k[4:], v[4:], beta[4:], g[4:], S1)
+    assert np.allclose(np.concatenate([o1, o2]), o) and np.allclose(S2, S)
+    ones = np.ones((3, 1, 4))
+    kk = np.repeat(O.unit(rng.standard_normal((1, 1, 4))), 3, axis=0)
+    o3, _ = O.delta_recurrence(kk, kk, v[:3, :1], np.ones((3, 1)), ones)
+    assert np.allclose(o3, v[:3, :1], atol=1e-5)          # full steps on one key: the last value replaces the one before
+    gz = np.ones((2, 1, 4)); gz[1, 0, 2] = 0.0
+    _, S4 = O.delta_recurrence(np.zeros((2, 1, 4)), np.stack([np.eye(4)[[2]], np.eye(4)[[0]]]), v[:2, :1], np.ones((2, 1)), gz)
+    assert np.allclose(S4[0, 2], 0.0) and np.allclose(S4[0, 0], v[1, 0])
+    u = rng.standard_normal((5, 2))
+    taps = np.array([[0.0, 0.0, 1.0], [1.0, 0.0, 0.0]])
+    c = O.conv_silu(u, taps)
+    assert np.allclose(c[:, 0], O.silu(u[:, 0])) and np.allclose(c[2:, 1], O.silu(u[:3, 1])) and np.allclose(c[:2, 1], 0.0)
+    tt = {n: np.asarray(x, np.float64) for n, x in w.items()}
+    h = tt["embed"][t]
+    y = O.attention(KAD_LEFT, tt, "l0.mix.left.", h, 1e-5)
+    hot = dict(tt); hot["l0.mix.left.sink"] = tt["l0.mix.left.sink"] + 60.0
+    assert np.abs(O.attention(KAD_LEFT, hot, "l0.mix.left.", h, 1e-5)).max() < 1e-12 * np.abs(y).max() + 1e-15
+    res = []
+    O.forward(cfg, w, t, res)
+    d = O.delta_rule(KAD_DELTA, tt, "l1.mix.", res[0], 1e-5)
+    assert np.allclose(res[1], res[0] + O.rms_norm(d, tt["l1.norm1"], 1e-5), atol=1e-12)
+
