@@ -183,7 +183,7 @@ struct LayeredEngine : nb::EngineBase {
     struct ResEpi { bool on = false; Dyt post{}, pre{}; float *out = nullptr, *keep = nullptr; } res;
     float *b_dpart = nullptr, *b_sseg = nullptr, *b_sdx = nullptr, *b_sdy = nullptr, *b_f2 = nullptr, *b_hg = nullptr, *b_sh2 = nullptr, *b_sg = nullptr, *b_wrow = nullptr; uint32_t *b_dtick = nullptr;
     // gated delta rule: convolved channels of a short portion; what the preparation hands the scan; low-rank products; outputs before and after the gate
-    float *b_gcv = nullptr, *b_gq = nullptr, *b_gk = nullptr, *b_gv = nullptr, *b_gg = nullptr, *b_gsc = nullptr, *b_gsp = nullptr, *b_gt = nullptr, *b_go = nullptr, *b_ga = nullptr;
+    float *b_gcv = nullptr, *b_gblk = nullptr, *b_gv = nullptr, *b_gsp = nullptr, *b_gt = nullptr, *b_go = nullptr, *b_ga = nullptr;
     float *b_gpart = nullptr; uint32_t *b_gtick = nullptr;      // grouped-query attention: partials and tickets of the key splits
     uint32_t *ids_dev = nullptr, *want_dev = nullptr, *next_dev = nullptr, *tok_host = nullptr; uint8_t *seen = nullptr;
     uint32_t last_T = 0;
@@ -773,15 +773,20 @@ int load_hc(Loader &ld, const std::string &p, uint32_t S, float **dst) {
 }
 
 // ---------------- launches ----------------
+// cluster: blocks per thread-block cluster along x (1: none)
 template <typename A>
-int launch(LayeredEngine *e, void (*k)(const A), dim3 grid, dim3 block, size_t smem, const A &args) {
+int launch(LayeredEngine *e, void (*k)(const A), dim3 grid, dim3 block, size_t smem, const A &args, uint32_t cluster = 1) {
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = grid; cfg.blockDim = block; cfg.dynamicSmemBytes = smem; cfg.stream = e->cur;
-    cudaLaunchAttribute attr[1];
+    cudaLaunchAttribute attr[2];
+    cfg.attrs = attr;
     if (e->use_pdl) {      // programmatic dependent launch: see pdl_enter() in layered_kernels.cuh
-        attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-        attr[0].val.programmaticStreamSerializationAllowed = 1;
-        cfg.attrs = attr; cfg.numAttrs = 1;
+        attr[cfg.numAttrs].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[cfg.numAttrs++].val.programmaticStreamSerializationAllowed = 1;
+    }
+    if (cluster > 1) {
+        attr[cfg.numAttrs].id = cudaLaunchAttributeClusterDimension;
+        attr[cfg.numAttrs].val.clusterDim.x = cluster; attr[cfg.numAttrs].val.clusterDim.y = 1; attr[cfg.numAttrs++].val.clusterDim.z = 1;
     }
     CK(cudaLaunchKernelEx(&cfg, k, args));
     e->launches++;
@@ -1211,9 +1216,9 @@ int delta_branch(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx
     if (T <= kGemvMaxM) {
         DeltaStepArgs a{e->b_gcv, e->b_p, P, L.c_b, L.c_a, L.c_g, L.ra ? L.a2.p : nullptr, L.rg ? L.g2.p : nullptr, L.ra, L.rg, L.d_bias, L.d_rate, L.d_gain,
                         cx.st + run.st_S, e->b_ga, T, H, G, D, VD, qscale, e->eps, e->f32 ? 0u : 1u};
-        const uint32_t want = std::max(128u, (VD + 3u) / 4u * 32u);
-#define DELTA_STEP(DCH) (e->f32 ? launch<DeltaStepArgs>(e, k_delta_step<float, DCH>, dim3(H), dim3(std::min(delta_step_threads(DCH), want)), delta_step_smem(DCH, VD), a) \
-                                : launch<DeltaStepArgs>(e, k_delta_step<__nv_bfloat16, DCH>, dim3(H), dim3(std::min(delta_step_threads(DCH), want)), delta_step_smem(DCH, VD), a))
+        const uint32_t nb = delta_step_blocks(VD), want = std::max(128u, delta_step_cols(VD) * 8u);
+#define DELTA_STEP(DCH) (e->f32 ? launch<DeltaStepArgs>(e, k_delta_step<float, DCH>, dim3(nb, H), dim3(std::min(kDeltaThreads, want)), delta_step_smem(DCH, VD), a, nb) \
+                                : launch<DeltaStepArgs>(e, k_delta_step<__nv_bfloat16, DCH>, dim3(nb, H), dim3(std::min(kDeltaThreads, want)), delta_step_smem(DCH, VD), a, nb))
         if (D <= 32) r = DELTA_STEP(1);
         else if (D <= 64) r = DELTA_STEP(2);
         else if (D <= 128) r = DELTA_STEP(4);
@@ -1225,14 +1230,14 @@ int delta_branch(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx
     if (L.rg && (r = gemm(e, plain(e->b_p + L.c_g, P, L.g2, e->b_gt, H * VD, T), 1, T))) return r;
     const uint32_t chunks = (T + kDeltaChunk - 1u) / kDeltaChunk;
     DeltaPrepArgs pa{e->b_p, P, L.c_conv, L.c_b, L.c_a, L.d_conv, cx.st + run.st_conv, L.d_taps, L.ra ? e->b_gsp : nullptr, L.d_bias, L.d_rate,
-                     e->b_gq, e->b_gk, e->b_gv, e->b_gg, e->b_gsc, T, H, G, D, VD, qscale};
-    if ((r = launch<DeltaPrepArgs>(e, k_delta_prep, dim3(chunks, H), dim3(32 * kDeltaChunk), 0, pa))) return r;
+                     e->b_gblk, e->b_gv, T, H, G, D, VD, qscale};
+    if ((r = launch<DeltaPrepArgs>(e, k_delta_prep, dim3(chunks, H), dim3(delta_dp(D)), 0, pa))) return r;
     if (L.d_taps > 1) {
         ConvArgs ca{e->b_p + L.c_conv, P, L.d_conv, nullptr, cx.st + run.st_conv, nullptr, T, C, L.d_taps, 0, 1};
         if ((r = launch<ConvArgs>(e, k_conv_state, dim3((C + 127u) / 128u), dim3(128), 0, ca))) return r;
     }
-    DeltaScanArgs sa{e->b_gq, e->b_gk, e->b_gv, e->b_gg, e->b_gsc, cx.st + run.st_S, e->b_go, T, H, G, D, VD, L.ra ? D : 1u};
-    const dim3 grid((VD + 15u) / 16u, H), block(128);
+    DeltaScanArgs sa{e->b_gblk, e->b_gv, cx.st + run.st_S, e->b_go, T, H, D, VD};
+    const dim3 grid((VD + 15u) / 16u, H), block(256);
     if (D <= 32) r = launch<DeltaScanArgs>(e, k_delta_scan<1>, grid, block, 0, sa);
     else if (D <= 64) r = launch<DeltaScanArgs>(e, k_delta_scan<2>, grid, block, 0, sa);
     else if (D <= 128) r = launch<DeltaScanArgs>(e, k_delta_scan<4>, grid, block, 0, sa);
@@ -2181,7 +2186,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
     uint32_t mC = 0, mZ = 0, mQR = 0, mQ = 0, mHR = 0, mOV = 0, mNE = 0, mTop = 0, mFF = 0, mSFF = 0;
     uint32_t sP = 0, sQK = 0, sXC = 0, sA = 0, sRO = 0, sDBC = 0, sF = 0;
     uint32_t sDP = 0, sDT = 0, sXC2 = 0, sY = 0, sF2 = 0; size_t sSS = 0, diff_smem[4] = {0, 0, 0, 0};      // differential attention, state-space duality, gated feed-forward
-    uint32_t dC = 0, dQ = 0, dV = 0, dGd = 0, dSc = 0, dSp = 0, dGt = 0, dPart = 0, dTick = 0; size_t gqa_smem[5] = {0, 0, 0, 0, 0};      // gated delta rule, grouped-query attention
+    uint32_t dC = 0, dV = 0, dBlk = 0, dSp = 0, dGt = 0, dPart = 0, dTick = 0; size_t gqa_smem[5] = {0, 0, 0, 0, 0};      // gated delta rule, grouped-query attention
     size_t win_smem[4] = {0, 0, 0, 0};      // most shared memory any layer asks of the window-attention instances, per value-column count
     for (const Run &q : e->runs) {
         const Layer &L = e->layers[q.layer];
@@ -2209,8 +2214,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
         }
         if (L.type == MIX_DELTA || L.type == MIX_ATTN_DELTA) {
             sP = std::max(sP, L.proj.rows);
-            dC = std::max(dC, 2 * L.dG * L.dD + L.dH * L.dVD); dQ = std::max(dQ, L.dG * L.dD); dV = std::max(dV, L.dH * L.dVD);
-            dGd = std::max(dGd, L.ra ? L.dH * L.dD : L.dH); dSc = std::max(dSc, L.dH * kDeltaSc);
+            dC = std::max(dC, 2 * L.dG * L.dD + L.dH * L.dVD); dV = std::max(dV, L.dH * L.dVD); dBlk = std::max(dBlk, L.dH * delta_block(delta_dp(L.dD)));
             if (L.ra) dSp = std::max(dSp, L.dH * L.dD);
             if (L.rg) dGt = std::max(dGt, L.dH * L.dVD);
         }
@@ -2232,8 +2236,8 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
         CK(cudaMemset(e->b_dtick, 0, (size_t)kGemvMaxM * sDT * 4));
     }
     if (dC) {
-        DM(e->b_gcv, (size_t)kGemvMaxM * dC * 4); DM(e->b_gq, T * dQ * 4); DM(e->b_gk, T * dQ * 4); DM(e->b_gv, T * dV * 4); DM(e->b_gg, T * dGd * 4);
-        DM(e->b_gsc, (T + kDeltaChunk - 1) / kDeltaChunk * dSc * 4); DM(e->b_go, T * dV * 4); DM(e->b_ga, T * dV * 4);
+        DM(e->b_gcv, (size_t)kGemvMaxM * dC * 4); DM(e->b_gv, T * dV * 4);
+        DM(e->b_gblk, (T + kDeltaChunk - 1) / kDeltaChunk * dBlk * 4); DM(e->b_go, T * dV * 4); DM(e->b_ga, T * dV * 4);
         if (dSp) DM(e->b_gsp, T * dSp * 4);
         if (dGt) DM(e->b_gt, T * dGt * 4);
     }

@@ -82,8 +82,7 @@ __global__ void __launch_bounds__(1024) k_post_norm(const PostNormArgs a) {
             x[i] = v;
             if (a.keep) a.keep[row + i] = v;
         }
-        return;
-    }
+    } else
     for (uint32_t i = threadIdx.x; i < a.E; i += blockDim.x) {
         const float u = d2 ? a.mix * (d[i] * ra * a.w1[i] + d2[i] * rb * a.w2[i]) : d[i];
         const float v = x[i] + u * rinv * a.w[i];
@@ -342,9 +341,13 @@ __global__ void __launch_bounds__(256) k_gqa_decode(const GqaArgs a) {
         }
     };
     fetch(tile_lo);
-    {   // root mean squares of the whole query row and, for a tail share, of the portion's key rows up to this token
-        float s[5] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
-        const uint32_t QW = a.H * D, KW = a.G * D;
+    // Norm factors are numbers per token: queries and keys are gained and turned without them (no wait for the sums), the scores and the
+    // cached key carry them.  red[0]: the whole query row's sum of squares; red[1 + u]: the key row's of the portion's token u (tail shares)
+    const uint32_t QW = a.H * D, KW = a.G * D;
+    {
+        float s[1 + kGemvMaxM];
+#pragma unroll
+        for (uint32_t u = 0; u <= kGemvMaxM; u++) s[u] = 0.0f;
         if (a.wq) {
             const float *q = a.p + (size_t)t * a.ld + a.q0;
             if (VEC) {
@@ -357,38 +360,45 @@ __global__ void __launch_bounds__(256) k_gqa_decode(const GqaArgs a) {
             for (uint32_t u = 0; u < kGemvMaxM; u++)
                 if (u <= t) { const float *k = a.p + (size_t)u * a.ld + a.k0; for (uint32_t i = tid; i < KW; i += 256u) s[1 + u] = fmaf(k[i], k[i], s[1 + u]); }
         }
-#pragma unroll
-        for (int j = 0; j < 5; j++) { s[j] = warp_sum(s[j]); if (lane == 0) red[j][warp] = s[j]; }
-        __syncthreads();
-        auto total = [&](uint32_t j) { float v = 0.0f; for (uint32_t w = 0; w < 8u; w++) v += red[j][w]; return v; };
-        const float rq = a.wq ? 1.0f / sqrtf(total(0) / (float)QW + a.eps) : 1.0f;
         for (uint32_t i = tid; i < nh * Dp; i += 256u) {
             const uint32_t h = i / Dp, d = i % Dp;
-            q_s[i] = d < D ? rot_half_at(a.p + (size_t)t * a.ld + a.q0 + (h0 + h) * D, a.wq ? a.wq + (h0 + h) * D : nullptr, rq, d, half, a.tab + (size_t)(pos + t) * half) * a.scale : 0.0f;
+            q_s[i] = d < D ? rot_half_at(a.p + (size_t)t * a.ld + a.q0 + (h0 + h) * D, a.wq ? a.wq + (h0 + h) * D : nullptr, 1.0f, d, half, a.tab + (size_t)(pos + t) * half) : 0.0f;
         }
-        for (uint32_t i = nh * Dp + tid; i < kGqaHeads * Dp; i += 256u) q_s[i] = 0.0f;
-        if (tail) {
-            float *row = a.cache + ((size_t)a.table[(pos + t) / kPage] * kPage + (pos + t) % kPage) * a.RL;
-            const bool own = split == nact - 1u && blockIdx.y % hgs == 0;      // one block writes the token's row of this key/value head
+        if (tail)
             for (uint32_t i = tid; i < (t + 1u) * Dp; i += 256u) {
                 const uint32_t u = i / Dp, d = i % Dp;
-                const float rk = a.wk ? 1.0f / sqrtf(total(1u + u) / (float)KW + a.eps) : 1.0f;
-                const float v = d < D ? rot_half_at(a.p + (size_t)u * a.ld + a.k0 + g * D, a.wk ? a.wk + g * D : nullptr, rk, d, half, a.tab + (size_t)(pos + u) * half) : 0.0f;
-                kn_s[i] = v;
-                if (own && u == t && d < D) row[g * D + d] = v;
+                kn_s[i] = d < D ? rot_half_at(a.p + (size_t)u * a.ld + a.k0 + g * D, a.wk ? a.wk + g * D : nullptr, 1.0f, d, half, a.tab + (size_t)(pos + u) * half) : 0.0f;
             }
-            if (own) for (uint32_t d = tid; d < VD; d += 256u) row[a.G * D + g * VD + d] = a.p[(size_t)t * a.ld + a.v0 + g * VD + d];
-        }
+#pragma unroll
+        for (uint32_t u = 0; u <= kGemvMaxM; u++) { s[u] = warp_sum(s[u]); if (lane == 0) red[u][warp] = s[u]; }
     }
     __syncthreads();
+    auto factor = [&](uint32_t j, bool normed, uint32_t n) {      // 1 / root mean square of row j of red
+        if (!normed) return 1.0f;
+        float v = 0.0f;
+#pragma unroll
+        for (uint32_t w = 0; w < 8u; w++) v += red[j][w];
+        return 1.0f / sqrtf(v / (float)n + a.eps);
+    };
+    const float qf = factor(0, a.wq != nullptr, QW) * a.scale;
+    if (split == nact - 1u && blockIdx.y % hgs == 0) {            // one block writes the token's row of this key/value head
+        float *row = a.cache + ((size_t)a.table[(pos + t) / kPage] * kPage + (pos + t) % kPage) * a.RL;
+        const float kf = factor(1u + t, a.wk != nullptr, KW);
+        for (uint32_t d = tid; d < D; d += 256u) row[g * D + d] = kn_s[t * Dp + d] * kf;
+        for (uint32_t d = tid; d < VD; d += 256u) row[a.G * D + g * VD + d] = a.p[(size_t)t * a.ld + a.v0 + g * VD + d];
+    }
     float o[CH], m = -INFINITY, l = 0.0f;              // o: items (head, column) tid, tid + 256, ...; m, l: of head `warp`
 #pragma unroll
     for (int c = 0; c < CH; c++) o[c] = 0.0f;
     for (uint32_t tile = tile_lo; tile < tile_hi; tile++) {
         const uint32_t kp = tile * kPage + key;
         if (kp >= pos && kp < nkeys) {
+            const float kf = factor(1u + kp - pos, a.wk != nullptr, KW);
 #pragma unroll
-            for (int c = 0; c < CH; c++) { const uint32_t d = (sub + 8u * c) * 4u; if (d < Dp) kr[c] = *reinterpret_cast<const float4 *>(kn_s + (kp - pos) * Dp + d); }
+            for (int c = 0; c < CH; c++) {
+                const uint32_t d = (sub + 8u * c) * 4u;
+                if (d < Dp) { const float4 v = *reinterpret_cast<const float4 *>(kn_s + (kp - pos) * Dp + d); kr[c] = make_float4(v.x * kf, v.y * kf, v.z * kf, v.w * kf); }
+            }
         }
         float acc[kGqaHeads];
 #pragma unroll
@@ -406,7 +416,7 @@ __global__ void __launch_bounds__(256) k_gqa_decode(const GqaArgs a) {
         for (uint32_t h = 0; h < kGqaHeads; h++) {
             if (h < nh) {
                 acc[h] += __shfl_xor_sync(0xffffffffu, acc[h], 4); acc[h] += __shfl_xor_sync(0xffffffffu, acc[h], 2); acc[h] += __shfl_xor_sync(0xffffffffu, acc[h], 1);
-                if (sub == h) s_s[h * kPage + key] = acc[h];
+                if (sub == h) s_s[h * kPage + key] = acc[h] * qf;
             }
         }
 #pragma unroll
@@ -523,10 +533,14 @@ __global__ void __launch_bounds__(256) k_gqa_decode(const GqaArgs a) {
 //     p_i = S^T (Gm_i k_i) + sum_{j<i} A_ij u_j,    A_ij = sum_d k_i k_j prod_{j<l<=i} g_l,    u_i = beta_i (v_i - p_i)
 //     o_i = S^T (Gm_i q_i) + sum_{j<=i} B_ij u_j,   B_ij = sum_d q_i k_j prod_{j<l<=i} g_l
 //     S  <- Gm_C S + sum_j (prod_{l>j} g_l k_j) u_j^T
-// so a value column meets its state twice per chunk instead of twice per token, and the sums over the key coordinates of all its
+// so  u = M_u w  and  o = S^T (Gm q) + M_o w  with  w_j = v_j - S^T (Gm_j k_j)  and two 4 x 4 triangular matrices made of A, B and beta alone:
+// a value column meets its state twice per chunk instead of twice per token, and the sums over the key coordinates of all its
 // tokens run side by side.  Every product of decays is a product of numbers in (0, 1], never a quotient.
 // ------------------------------------------------------------------------------------------------
-constexpr uint32_t kDeltaChunk = 4, kDeltaDim = 256, kDeltaSc = 36;      // kDeltaSc: floats per (chunk, head): A [4][4], B [4][4], beta [4]
+constexpr uint32_t kDeltaChunk = 4, kDeltaDim = 256, kDeltaVecs = 3 * kDeltaChunk + 1, kDeltaMat = 2 * kDeltaChunk * kDeltaChunk;
+// what the scan reads of a chunk and head, in one run: Gm_i k_i (4), Gm_i q_i (4), prod_{l>j} g_l k_j (4), Gm_C, each `dp` coordinates; M_u, M_o
+__host__ __device__ inline uint32_t delta_dp(uint32_t D) { return D <= 32u ? 32u : D <= 64u ? 64u : D <= 128u ? 128u : 256u; }
+__host__ __device__ inline uint32_t delta_block(uint32_t dp) { return kDeltaVecs * dp + kDeltaMat; }
 // exp(-rate sp), in double precision and rounded once: a state that forgets slowly takes thousands of these factors
 __device__ __forceinline__ float delta_decay(float rate, float sp) { return (float)exp(-(double)rate * (double)sp); }
 
@@ -534,220 +548,271 @@ struct DeltaPrepArgs {
     const float *p; uint32_t ld, c0, b0, a0; const float *taps; const float *state; uint32_t K;      // c0: the first convolved channel's column
     const float *sp;                       // per-channel decay: softplus already taken, [T][H D]; null: one decay per head from column a0 + h
     const float *dt_bias, *rate;
-    float *q, *k, *v, *g, *sc;             // q, k [T][G D], v [T][H VD], g [T][H D] (or [T][H]), sc [chunks][H][kDeltaSc]
+    float *blk, *v;                        // blk [chunks][H][delta_block], v [T][H VD]
     uint32_t T, H, G, D, VD; float qscale;
 };
-// grid = (chunks, heads); a warp per token of the chunk
-__global__ void __launch_bounds__(32 * kDeltaChunk) k_delta_prep(const DeltaPrepArgs a) {
+// grid = (chunks, heads), delta_dp(D) threads: a thread makes the chunk's tokens of its key coordinate (and of some value columns).  All sums
+// over the coordinates -- squares, and the products between tokens -- are taken of the vectors before they become unit vectors, in one
+// reduction; their factors join afterwards.
+__global__ void __launch_bounds__(kDeltaDim) k_delta_prep(const DeltaPrepArgs a) {
     pdl_enter();
-    __shared__ float q_s[kDeltaChunk][kDeltaDim], k_s[kDeltaChunk][kDeltaDim], g_s[kDeltaChunk][kDeltaDim];
-    const uint32_t w = threadIdx.x >> 5, lane = threadIdx.x & 31u, t = blockIdx.x * kDeltaChunk + w, h = blockIdx.y, rep = a.H / a.G, g = h / rep;
-    const uint32_t D = a.D, GD = a.G * D, C = 2u * GD + a.H * a.VD;
-    float *sc = a.sc + ((size_t)blockIdx.x * a.H + h) * kDeltaSc;
-    if (t < a.T) {
-        auto conv = [&](uint32_t c) {
-            float s = 0.0f;
-            for (uint32_t j = 0; j < a.K; j++) {
-                const int32_t src = (int32_t)t - (int32_t)(a.K - 1u - j);
-                s = fmaf(a.taps[(size_t)c * a.K + j], src >= 0 ? a.p[(size_t)src * a.ld + a.c0 + c] : a.state[(size_t)((int32_t)(a.K - 1u) + src) * C + c], s);
-            }
-            return siluf_(s);
-        };
-        float sq = 0.0f, sk = 0.0f;
-        for (uint32_t d = lane; d < D; d += 32u) {
-            const float qv = conv(g * D + d), kv = conv(GD + g * D + d);
-            q_s[w][d] = qv; k_s[w][d] = kv;
-            sq = fmaf(qv, qv, sq); sk = fmaf(kv, kv, sk);
-        }
-        const float rq = a.qscale / sqrtf(warp_sum(sq) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(sk) + 1e-6f), rate = a.rate[h];
-        float gh = 1.0f;
-        if (!a.sp) {
-            gh = delta_decay(rate, softplusf_(a.p[(size_t)t * a.ld + a.a0 + h] + a.dt_bias[h]));
-            if (lane == 0) a.g[(size_t)t * a.H + h] = gh;
-        }
-        for (uint32_t d = lane; d < D; d += 32u) {
-            const float qv = q_s[w][d] * rq, kv = k_s[w][d] * rk;
-            q_s[w][d] = qv; k_s[w][d] = kv;
-            if (h % rep == 0) { a.q[(size_t)t * GD + g * D + d] = qv; a.k[(size_t)t * GD + g * D + d] = kv; }
-            float gv = gh;
-            if (a.sp) { const size_t at = ((size_t)t * a.H + h) * D + d; gv = delta_decay(rate, a.sp[at]); a.g[at] = gv; }
-            g_s[w][d] = gv;
-        }
-        for (uint32_t j = lane; j < a.VD; j += 32u) a.v[(size_t)t * a.H * a.VD + h * a.VD + j] = conv(2u * GD + h * a.VD + j);
-        if (lane == 0) sc[32u + w] = sigmoidf_(a.p[(size_t)t * a.ld + a.b0 + h]);
-    } else {                               // tokens past the portion: nothing is forgotten, nothing is written
-        for (uint32_t d = lane; d < D; d += 32u) { q_s[w][d] = 0.0f; k_s[w][d] = 0.0f; g_s[w][d] = 1.0f; }
-        if (lane == 0) sc[32u + w] = 0.0f;
-    }
-    __syncthreads();
-    float A[kDeltaChunk], B[kDeltaChunk];      // row i = w
+    constexpr uint32_t C4 = kDeltaChunk;
+    __shared__ float red[8][32], tot[32], fac[2 * C4], beta_s[C4];
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, nw = blockDim.x >> 5, DP = blockDim.x, t0 = blockIdx.x * C4, h = blockIdx.y, g = h / (a.H / a.G);
+    const uint32_t D = a.D, GD = a.G * D, C = 2u * GD + a.H * a.VD, K = a.K;
+    float *blk = a.blk + ((size_t)blockIdx.x * a.H + h) * delta_block(DP);
+    // one row of channel c before (or in) the portion
+    auto input = [&](int32_t src, uint32_t c) {
+        return src >= 0 ? (src < (int32_t)a.T ? a.p[(size_t)src * a.ld + a.c0 + c] : 0.0f) : a.state[(size_t)((int32_t)(K - 1u) + src) * C + c];
+    };
+    float q[C4], k[C4], gv[C4];
 #pragma unroll
-    for (uint32_t j = 0; j < kDeltaChunk; j++) { A[j] = 0.0f; B[j] = 0.0f; }
-    for (uint32_t d = lane; d < D; d += 32u) {
-        const float kv = k_s[w][d], qv = q_s[w][d];
+    for (uint32_t i = 0; i < C4; i++) { q[i] = 0.0f; k[i] = 0.0f; gv[i] = 1.0f; }
+    const float rate = a.rate[h];
+    if (tid < D) {
+        const uint32_t cq = g * D + tid, ck = GD + cq;
+        float wq[C4], wk[C4];              // the taps that meet input m for tokens 0..3: taps[m - i]
+#pragma unroll
+        for (uint32_t i = 0; i < C4; i++) { wq[i] = 0.0f; wk[i] = 0.0f; }
+#pragma unroll 4
+        for (uint32_t m = 0; m < K + C4 - 1u; m++) {
+            const int32_t src = (int32_t)(t0 + m) - (int32_t)(K - 1u);
+            const float xq = input(src, cq), xk = input(src, ck);
+#pragma unroll
+            for (int i = (int)C4 - 1; i > 0; i--) { wq[i] = wq[i - 1]; wk[i] = wk[i - 1]; }
+            wq[0] = m < K ? a.taps[(size_t)cq * K + m] : 0.0f; wk[0] = m < K ? a.taps[(size_t)ck * K + m] : 0.0f;
+#pragma unroll
+            for (uint32_t i = 0; i < C4; i++) { q[i] = fmaf(wq[i], xq, q[i]); k[i] = fmaf(wk[i], xk, k[i]); }
+        }
+#pragma unroll
+        for (uint32_t i = 0; i < C4; i++) {
+            const uint32_t t = t0 + i;
+            if (t < a.T) {
+                q[i] = siluf_(q[i]); k[i] = siluf_(k[i]);
+                gv[i] = delta_decay(rate, a.sp ? a.sp[((size_t)t * a.H + h) * D + tid] : softplusf_(a.p[(size_t)t * a.ld + a.a0 + h] + a.dt_bias[h]));
+            } else { q[i] = 0.0f; k[i] = 0.0f; }      // tokens past the portion: nothing is forgotten, nothing is written
+        }
+    }
+    if (tid < C4) beta_s[tid] = t0 + tid < a.T ? sigmoidf_(a.p[(size_t)(t0 + tid) * a.ld + a.b0 + h]) : 0.0f;
+    // sums 0..3: q_i^2, 4..7: k_i^2, 8 + i (i - 1) / 2 + j: k_i k_j prod_{j<l<=i} g_l (j < i), 14 + i (i + 1) / 2 + j: q_i k_j prod (j <= i)
+    float x[32];
+#pragma unroll
+    for (int i = 0; i < 32; i++) x[i] = 0.0f;
+#pragma unroll
+    for (int i = 0; i < (int)C4; i++) {
+        x[i] = q[i] * q[i]; x[4 + i] = k[i] * k[i];
         float dec = 1.0f;
 #pragma unroll
-        for (int j = (int)kDeltaChunk - 1; j >= 0; j--) {
-            if (j > (int)w) continue;
-            if (j < (int)w) { dec *= g_s[j + 1][d]; A[j] = fmaf(kv * dec, k_s[j][d], A[j]); }
-            B[j] = fmaf(qv * dec, k_s[j][d], B[j]);
+        for (int j = i; j >= 0; j--) {
+            if (j < i) { dec *= gv[j + 1]; x[8 + i * (i - 1) / 2 + j] = k[i] * k[j] * dec; }
+            x[14 + i * (i + 1) / 2 + j] = q[i] * k[j] * dec;
         }
     }
+    // 32 sums over 32 lanes: lane l ends with sum l
 #pragma unroll
-    for (uint32_t j = 0; j < kDeltaChunk; j++) {
-        const float x = warp_sum(A[j]), y = warp_sum(B[j]);
-        if (lane == 0) { sc[w * 4u + j] = x; sc[16u + w * 4u + j] = y; }
-    }
-}
-
-// A block of 4 warps owns 16 value columns of head h = blockIdx.y; 8 lanes share a column (lane s holds coordinates 4 s + 32 c .. + 3).
-// The chunk vectors Gm_i k_i, Gm_i q_i, prod_{l>j} g_l k_j and Gm_C are made while a tile of NCH chunks is staged; the tile after it is
-// in flight (registers) meanwhile.
-struct DeltaScanArgs { const float *q, *k, *v, *g, *sc; float *S; float *o; uint32_t T, H, G, D, VD, gdim; };      // gdim: decays per head (D or 1)
-template <int DCH>
-__global__ void __launch_bounds__(128) k_delta_scan(const DeltaScanArgs a) {
-    pdl_enter();
-    constexpr uint32_t DP = DCH * 32u, NCH = DCH <= 4 ? 2u : 1u, NI = (NCH * DP + 127u) / 128u, NVEC = 3u * kDeltaChunk + 1u;
-    __shared__ __align__(16) float w_s[2][NCH][NVEC][DP], v_s[2][NCH][16][4], c_s[2][NCH][kDeltaSc];
-    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, sub = lane & 7u, cl = warp * 4u + (lane >> 3), h = blockIdx.y, col0 = blockIdx.x * 16u, col = col0 + cl;
-    const uint32_t D = a.D, GD = a.G * D, HV = a.H * a.VD, gk = (h / (a.H / a.G)) * D;
-    const bool dvec = (D & 3u) == 0;
-    float *Sp = a.S + ((size_t)h * a.VD + col) * D;
-    float S[DCH][4];
+    for (int half = 16; half > 0; half >>= 1) {
+        const bool up = lane & half;
 #pragma unroll
-    for (int c = 0; c < DCH; c++) {
-        const uint32_t d = (sub + 8u * c) * 4u;
-#pragma unroll
-        for (int e = 0; e < 4; e++) S[c][e] = 0.0f;
-        if (col < a.VD && d < D) {
-            if (dvec) { const float4 v = *reinterpret_cast<const float4 *>(Sp + d); S[c][0] = v.x; S[c][1] = v.y; S[c][2] = v.z; S[c][3] = v.w; }
-            else {
-#pragma unroll
-                for (uint32_t e = 0; e < 4; e++) if (d + e < D) S[c][e] = Sp[d + e];
-            }
+        for (int i = 0; i < half; i++) {
+            const float keep = up ? x[i + half] : x[i], give = up ? x[i] : x[i + half];
+            x[i] = keep + __shfl_xor_sync(0xffffffffu, give, half);
         }
     }
-    float rk[NI][4], rq[NI][4], rg[NI][4], rv = 0.0f, rc = 0.0f;
-    auto fetch = [&](uint32_t ch0) {           // the tile that starts at chunk ch0
+    red[warp][lane] = x[0];
+    // the value columns, meanwhile
+    for (uint32_t j = tid; j < a.VD; j += blockDim.x) {
+        const uint32_t cv = 2u * GD + h * a.VD + j;
+        float v[C4], wv[C4];
 #pragma unroll
-        for (uint32_t n = 0; n < NI; n++) {
-            const uint32_t it = tid + 128u * n, c = it / DP, d = it % DP;
+        for (uint32_t i = 0; i < C4; i++) { v[i] = 0.0f; wv[i] = 0.0f; }
+#pragma unroll 4
+        for (uint32_t m = 0; m < K + C4 - 1u; m++) {
+            const float xv = input((int32_t)(t0 + m) - (int32_t)(K - 1u), cv);
 #pragma unroll
-            for (uint32_t i = 0; i < kDeltaChunk; i++) {
-                const uint32_t t = (ch0 + c) * kDeltaChunk + i;
-                const bool ok = c < NCH && t < a.T && d < D;
-                rk[n][i] = ok ? __ldg(a.k + (size_t)t * GD + gk + d) : 0.0f;
-                rq[n][i] = ok ? __ldg(a.q + (size_t)t * GD + gk + d) : 0.0f;
-                rg[n][i] = ok ? __ldg(a.g + ((size_t)t * a.H + h) * a.gdim + (a.gdim > 1u ? d : 0u)) : 1.0f;
-            }
+            for (int i = (int)C4 - 1; i > 0; i--) wv[i] = wv[i - 1];
+            wv[0] = m < K ? a.taps[(size_t)cv * K + m] : 0.0f;
+#pragma unroll
+            for (uint32_t i = 0; i < C4; i++) v[i] = fmaf(wv[i], xv, v[i]);
         }
-        {
-            const uint32_t c = tid / 64u, i = (tid / 16u) % 4u, j = col0 + tid % 16u, t = (ch0 + c) * kDeltaChunk + i;
-            rv = (c < NCH && t < a.T && j < a.VD) ? __ldg(a.v + (size_t)t * HV + h * a.VD + j) : 0.0f;
-        }
-        const uint32_t c = tid / kDeltaSc;
-        rc = (c < NCH && (ch0 + c) * kDeltaChunk < a.T) ? __ldg(a.sc + ((size_t)(ch0 + c) * a.H + h) * kDeltaSc + tid % kDeltaSc) : 0.0f;
-    };
-    auto stage = [&](uint32_t b) {
 #pragma unroll
-        for (uint32_t n = 0; n < NI; n++) {
-            const uint32_t it = tid + 128u * n, c = it / DP, d = it % DP;
-            if (c >= NCH) continue;
-            float pre = 1.0f, suf = 1.0f;
-#pragma unroll
-            for (uint32_t i = 0; i < kDeltaChunk; i++) { pre *= rg[n][i]; w_s[b][c][i][d] = pre * rk[n][i]; w_s[b][c][kDeltaChunk + i][d] = pre * rq[n][i]; }
-            w_s[b][c][3u * kDeltaChunk][d] = pre;
-#pragma unroll
-            for (int i = (int)kDeltaChunk - 1; i >= 0; i--) { w_s[b][c][2u * kDeltaChunk + i][d] = suf * rk[n][i]; suf *= rg[n][i]; }
-        }
-        if (tid / 64u < NCH) v_s[b][tid / 64u][tid % 16u][(tid / 16u) % 4u] = rv;
-        if (tid / kDeltaSc < NCH) c_s[b][tid / kDeltaSc][tid % kDeltaSc] = rc;
-    };
-    const uint32_t chunks = (a.T + kDeltaChunk - 1u) / kDeltaChunk;
-    fetch(0);
-    stage(0);
+        for (uint32_t i = 0; i < C4; i++) if (t0 + i < a.T) a.v[(size_t)(t0 + i) * a.H * a.VD + h * a.VD + j] = siluf_(v[i]);
+    }
     __syncthreads();
-    uint32_t b = 0;
-    for (uint32_t ch0 = 0; ch0 < chunks; ch0 += NCH, b ^= 1u) {
-        if (ch0 + NCH < chunks) fetch(ch0 + NCH);
-#pragma unroll 1
-        for (uint32_t c = 0; c < NCH && ch0 + c < chunks; c++) {
-            const float *w = &w_s[b][c][0][0];
-            float x[8];                        // 0..3: S^T (Gm_i k_i), 4..7: S^T (Gm_i q_i)
-#pragma unroll
-            for (int i = 0; i < 8; i++) x[i] = 0.0f;
-#pragma unroll
-            for (int cc = 0; cc < DCH; cc++) {
-                const uint32_t d = (sub + 8u * cc) * 4u;
-#pragma unroll
-                for (int i = 0; i < 8; i++) {
-                    const float4 f = *reinterpret_cast<const float4 *>(w + i * DP + d);
-                    x[i] = fmaf(S[cc][3], f.w, fmaf(S[cc][2], f.z, fmaf(S[cc][1], f.y, fmaf(S[cc][0], f.x, x[i]))));
-                }
-            }
-            // eight sums over eight lanes with seven shuffles: lane s ends with sum s
-            const bool b4 = sub & 4u, b2 = sub & 2u, b1 = sub & 1u;
-            float y4[4], y2[2], mine;
-#pragma unroll
-            for (int i = 0; i < 4; i++) y4[i] = (b4 ? x[i + 4] : x[i]) + __shfl_xor_sync(0xffffffffu, b4 ? x[i] : x[i + 4], 4);
-#pragma unroll
-            for (int i = 0; i < 2; i++) y2[i] = (b2 ? y4[i + 2] : y4[i]) + __shfl_xor_sync(0xffffffffu, b2 ? y4[i] : y4[i + 2], 2);
-            mine = (b1 ? y2[1] : y2[0]) + __shfl_xor_sync(0xffffffffu, b1 ? y2[0] : y2[1], 1);
-            const float *sc = c_s[b][c];
-            const float4 vv = *reinterpret_cast<const float4 *>(v_s[b][c][cl]);
-            const float vi[4] = {vv.x, vv.y, vv.z, vv.w};
-            float u[4];
-#pragma unroll
-            for (int i = 0; i < 4; i++) {
-                float p = __shfl_sync(0xffffffffu, mine, (lane & 24u) + i);
-#pragma unroll
-                for (int j = 0; j < i; j++) p = fmaf(sc[i * 4 + j], u[j], p);
-                u[i] = sc[32 + i] * (vi[i] - p);
-            }
-            if (b4) {                          // lanes 4..7 of a column write token 0..3's output (B_ij is zero for j > i)
-                const uint32_t i = sub & 3u, t = (ch0 + c) * kDeltaChunk + i;
-                float o = mine;
-#pragma unroll
-                for (int j = 0; j < 4; j++) o = fmaf(sc[16 + i * 4 + j], u[j], o);
-                if (t < a.T && col < a.VD) a.o[(size_t)t * HV + h * a.VD + col] = o;
-            }
-#pragma unroll
-            for (int cc = 0; cc < DCH; cc++) {
-                const uint32_t d = (sub + 8u * cc) * 4u;
-                const float4 f = *reinterpret_cast<const float4 *>(w + 12 * DP + d);
-                S[cc][0] *= f.x; S[cc][1] *= f.y; S[cc][2] *= f.z; S[cc][3] *= f.w;
-#pragma unroll
-                for (int j = 0; j < 4; j++) {
-                    const float4 kk = *reinterpret_cast<const float4 *>(w + (8 + j) * DP + d);
-                    S[cc][0] = fmaf(kk.x, u[j], S[cc][0]); S[cc][1] = fmaf(kk.y, u[j], S[cc][1]); S[cc][2] = fmaf(kk.z, u[j], S[cc][2]); S[cc][3] = fmaf(kk.w, u[j], S[cc][3]);
-                }
-            }
-        }
-        if (ch0 + NCH < chunks) stage(b ^ 1u);
-        __syncthreads();
+    if (tid < 32u) {
+        float s = 0.0f;
+        for (uint32_t w = 0; w < nw; w++) s += red[w][tid];
+        tot[tid] = s;
+        if (tid < 2u * C4) fac[tid] = (tid < C4 ? a.qscale : 1.0f) / sqrtf(s + 1e-6f);      // the unit vectors' factors: q 0..3, k 4..7
     }
+    __syncthreads();
+    {
+        float pre = 1.0f, suf = 1.0f;
 #pragma unroll
-    for (int c = 0; c < DCH; c++) {
-        const uint32_t d = (sub + 8u * c) * 4u;
-        if (col < a.VD && d < D) {
-            if (dvec) *reinterpret_cast<float4 *>(Sp + d) = make_float4(S[c][0], S[c][1], S[c][2], S[c][3]);
-            else {
+        for (uint32_t i = 0; i < C4; i++) {
+            pre *= gv[i];
+            k[i] *= fac[C4 + i];
+            blk[i * DP + tid] = pre * k[i];
+            blk[(C4 + i) * DP + tid] = pre * (q[i] * fac[i]);
+        }
 #pragma unroll
-                for (uint32_t e = 0; e < 4; e++) if (d + e < D) Sp[d + e] = S[c][e];
-            }
+        for (int i = (int)C4 - 1; i >= 0; i--) { blk[(2u * C4 + i) * DP + tid] = suf * k[i]; suf *= gv[i]; }
+        blk[3u * C4 * DP + tid] = pre;
+    }
+    // w = v - S^T (Gm k)  ->  u = M_u w with rows M_i = beta_i (e_i - sum_{j<i} A_ij M_j), and o = S^T (Gm q) + (B M_u) w: column `tid` of both
+    if (tid < C4) {
+        float M[C4], *mat = blk + kDeltaVecs * DP;
+#pragma unroll
+        for (int i = 0; i < (int)C4; i++) {
+            float v = i == (int)tid ? 1.0f : 0.0f;
+#pragma unroll
+            for (int j = 0; j < i; j++) v = fmaf(-tot[8 + i * (i - 1) / 2 + j] * fac[C4 + i] * fac[C4 + j], M[j], v);
+            M[i] = beta_s[i] * v;
+            mat[i * C4 + tid] = M[i];
+        }
+#pragma unroll
+        for (int i = 0; i < (int)C4; i++) {
+            float v = 0.0f;
+#pragma unroll
+            for (int j = 0; j <= i; j++) v = fmaf(tot[14 + i * (i + 1) / 2 + j] * fac[i] * fac[C4 + j], M[j], v);
+            mat[C4 * C4 + i * C4 + tid] = v;
         }
     }
 }
 
-// Short portions (T <= kGemvMaxM): one block per head, from the convolved channels (an epilogue of the joint product) to the normed and
-// gated output.  8 lanes share a value column.  Low-rank decay and gate: their second products, W_a2 (a1) and W_g2 (g1) with a1, g1
+// A block of 8 warps owns 16 value columns of head h = blockIdx.y, a warp two of them; the 32 lanes share the key coordinates.  A chunk
+// takes 8 sums over the coordinates per column (four S^T (Gm_i k_i), four S^T (Gm_i q_i)); the warp reduces its 16 sums with 16 shuffles
+// and no selection, because lane l keeps sum (i, column c) in the place (i ^ (l / 4), c ^ (l / 2 % 2)) from the start -- it reads the chunk
+// vectors in that order and its two columns of the state sit in that order.  Lanes 2 n and 2 n + 1 end with sum n.  Tiles of NCH chunks
+// travel two ahead (cp.async into a ring of three).
+struct DeltaScanArgs { const float *blk, *v; float *S; float *o; uint32_t T, H, D, VD; };
+template <int VW> __device__ __forceinline__ void lds_vec(const float *p, float *v) {
+    if constexpr (VW == 4) { const float4 f = *reinterpret_cast<const float4 *>(p); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+    else if constexpr (VW == 2) { const float2 f = *reinterpret_cast<const float2 *>(p); v[0] = f.x; v[1] = f.y; }
+    else v[0] = *p;
+}
+__device__ __forceinline__ void cp_async4(float *dst, const float *src, bool ok) {      // 4 bytes into shared memory; zero when !ok
+    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst), n = ok ? 4u : 0u;
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(d), "l"(src), "r"(n) : "memory");
+}
+template <int DCH>
+__global__ void __launch_bounds__(256, 2) k_delta_scan(const DeltaScanArgs a) {
+    pdl_enter();
+    constexpr uint32_t DP = DCH * 32u, NCH = DCH <= 4 ? 2u : 1u, BLK = kDeltaVecs * DP + kDeltaMat;
+    constexpr int VW = DCH < 4 ? DCH : 4, NB = DCH / VW;      // a lane's coordinates: NB runs of VW, at (run * 32 + lane) * VW
+    __shared__ __align__(16) float w_s[3][NCH][BLK];
+    __shared__ __align__(16) float v_s[3][NCH][4][16];
+    __shared__ __align__(16) float u_s[8][2][2][4];
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, li = lane >> 2, lc = (lane >> 1) & 1u, h = blockIdx.y, col0 = blockIdx.x * 16u, jw = col0 + warp * 2u;
+    const uint32_t D = a.D, HV = a.H * a.VD, chunks = (a.T + kDeltaChunk - 1u) / kDeltaChunk, tiles = (chunks + NCH - 1u) / NCH;
+    auto fetch = [&](uint32_t tile) {          // one group of copies per tile, an empty one past the last
+        if (tile < tiles) {
+            const uint32_t st = tile % 3u, ch0 = tile * NCH;
+            for (uint32_t i = tid; i < NCH * (BLK / 4u); i += 256u) {
+                const uint32_t c = i / (BLK / 4u), e = (i % (BLK / 4u)) * 4u;
+                if (ch0 + c < chunks) cp_async16(&w_s[st][c][e], a.blk + ((size_t)(ch0 + c) * a.H + h) * BLK + e, true);
+            }
+            if (tid < NCH * 64u) {
+                const uint32_t c = tid / 64u, i = (tid / 16u) % 4u, j = tid % 16u, t = (ch0 + c) * kDeltaChunk + i;
+                const bool ok = t < a.T && col0 + j < a.VD;
+                cp_async4(&v_s[st][c][i][j], ok ? a.v + (size_t)t * HV + h * a.VD + col0 + j : a.v, ok);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch(0); fetch(1);
+    float S[2][DCH];                           // S[c]: column jw + (c ^ lc)
+#pragma unroll
+    for (uint32_t c = 0; c < 2; c++)
+#pragma unroll
+        for (int e = 0; e < DCH; e++) {
+            const uint32_t d = ((e / VW) * 32u + lane) * VW + e % VW, col = jw + (c ^ lc);
+            S[c][e] = (col < a.VD && d < D) ? a.S[((size_t)h * a.VD + col) * D + d] : 0.0f;
+        }
+    for (uint32_t tile = 0; tile < tiles; tile++) {
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();                       // this tile has landed for every thread, and the one before is done with: its place is free
+        fetch(tile + 2u);
+        const uint32_t st = tile % 3u;
+#pragma unroll
+        for (uint32_t c = 0; c < NCH; c++) {
+            if (tile * NCH + c >= chunks) break;
+            const float *w = &w_s[st][c][lane * VW], *mat = &w_s[st][c][kDeltaVecs * DP];
+            float x[8][2];
+#pragma unroll
+            for (uint32_t i = 0; i < 8; i++) {
+                float f[DCH];
+#pragma unroll
+                for (int n = 0; n < NB; n++) lds_vec<VW>(w + (i ^ li) * DP + n * 32 * VW, f + n * VW);
+#pragma unroll
+                for (int j = 0; j < 2; j++) {
+                    x[i][j] = S[j][0] * f[0];
+#pragma unroll
+                    for (int e = 1; e < DCH; e++) x[i][j] = fmaf(S[j][e], f[e], x[i][j]);
+                }
+            }
+#pragma unroll
+            for (int half = 4; half > 0; half >>= 1)
+#pragma unroll
+                for (int i = 0; i < half; i++)
+#pragma unroll
+                    for (int j = 0; j < 2; j++) x[i][j] += __shfl_xor_sync(0xffffffffu, x[i + half][j], half * 4);
+            float mine = x[0][0] + __shfl_xor_sync(0xffffffffu, x[0][1], 2);
+            mine += __shfl_xor_sync(0xffffffffu, mine, 1);      // lanes 0..15: S^T (Gm_i k_i), 16..31: S^T (Gm_i q_i), i = li % 4, column jw + lc
+            const float wj = v_s[st][c][li & 3u][warp * 2u + lc] - mine;
+            const float4 mr = *reinterpret_cast<const float4 *>(mat + li * 4u);
+            float y = li < 4u ? 0.0f : mine;
+            y = fmaf(mr.x, __shfl_sync(0xffffffffu, wj, lc * 2u), y); y = fmaf(mr.y, __shfl_sync(0xffffffffu, wj, 4u + lc * 2u), y);
+            y = fmaf(mr.z, __shfl_sync(0xffffffffu, wj, 8u + lc * 2u), y); y = fmaf(mr.w, __shfl_sync(0xffffffffu, wj, 12u + lc * 2u), y);
+            if ((lane & 1u) == 0) {
+                if (li < 4u) u_s[warp][c & 1u][lc][li] = y;
+                else {
+                    const uint32_t t = (tile * NCH + c) * kDeltaChunk + (li & 3u);
+                    if (t < a.T && jw + lc < a.VD) a.o[(size_t)t * HV + h * a.VD + jw + lc] = y;
+                }
+            }
+            float f[5][DCH];                   // the writes' keys, decayed to the chunk's end, and the chunk's whole decay
+#pragma unroll
+            for (int i = 0; i < 5; i++)
+#pragma unroll
+                for (int n = 0; n < NB; n++) lds_vec<VW>(w + (8 + i) * DP + n * 32 * VW, f[i] + n * VW);
+            __syncwarp();
+            float u[2][4];                     // u[c]: the four tokens' steps of column jw + (c ^ lc)
+#pragma unroll
+            for (uint32_t j = 0; j < 2; j++) lds_vec<4>(&u_s[warp][c & 1u][j ^ lc][0], u[j]);
+#pragma unroll
+            for (int j = 0; j < 2; j++)
+#pragma unroll
+                for (int e = 0; e < DCH; e++) {
+                    float v = S[j][e] * f[4][e];
+#pragma unroll
+                    for (int i = 0; i < 4; i++) v = fmaf(f[i][e], u[j][i], v);
+                    S[j][e] = v;
+                }
+        }
+    }
+    asm volatile("cp.async.wait_all;" ::: "memory");
+#pragma unroll
+    for (uint32_t c = 0; c < 2; c++)
+#pragma unroll
+        for (int e = 0; e < DCH; e++) {
+            const uint32_t d = ((e / VW) * 32u + lane) * VW + e % VW, col = jw + (c ^ lc);
+            if (col < a.VD && d < D) a.S[((size_t)h * a.VD + col) * D + d] = S[c][e];
+        }
+}
+
+// Short portions (T <= kGemvMaxM): a cluster of blocks per head, each with a share of its value columns, from the convolved channels (an
+// epilogue of the joint product) to the normed and gated output; the blocks exchange their columns' sums of squares through each other's
+// shared memory.  8 lanes share a value column.  Low-rank decay and gate: their second products, W_a2 (a1) and W_g2 (g1) with a1, g1
 // columns of the joint product, are made here for the head's own rows (round_a: the operand rounded to bf16 first, as a tensor-core
 // product would).  Without them the decay is one number per head (column a0 + h) and the gate silu of H VD columns at g0.
+constexpr uint32_t kDeltaBlocks = 4;       // blocks per head at most
+__host__ __device__ inline uint32_t delta_step_blocks(uint32_t VD) { return VD >= 64u ? 4u : VD >= 32u ? 2u : 1u; }
+__host__ __device__ inline uint32_t delta_step_cols(uint32_t VD) { const uint32_t n = delta_step_blocks(VD); return ((VD + n - 1u) / n + 3u) & ~3u; }
 struct DeltaStepArgs {
     const float *cv; const float *p; uint32_t ld, b0, a0, g0; const void *a2, *g2; uint32_t ra, rg; const float *dt_bias, *rate, *gain;
     float *S; float *out; uint32_t T, H, G, D, VD; float qscale, eps; uint32_t round_a;
 };
-inline size_t delta_step_smem(int dch, uint32_t VD) { return ((size_t)3 * kGemvMaxM * (uint32_t)dch * 32u + (size_t)2 * kGemvMaxM * VD) * 4; }      // dch: the instance's, DCH
+inline size_t delta_step_smem(int dch, uint32_t VD) { return ((size_t)3 * kGemvMaxM * (uint32_t)dch * 32u + (size_t)2 * kGemvMaxM * delta_step_cols(VD)) * 4; }      // dch: the instance's, DCH
 // dot products of one weight row with up to kGemvMaxM rows of x (stride ld), 8 lanes per row; every lane gets the totals.  vec: 16-byte
 // loads of both operands are aligned
 template <typename WT>
@@ -779,30 +844,40 @@ __device__ __forceinline__ void lane8_dots(const WT *w, const float *x, uint32_t
 #pragma unroll
     for (uint32_t t = 0; t < kGemvMaxM; t++) { acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], 4); acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], 2); acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], 1); }
 }
-constexpr uint32_t delta_step_threads(int dch) { return dch <= 4 ? 1024u : 512u; }
+constexpr uint32_t kDeltaThreads = 512;    // a block's threads at most (8 per value column; more columns: several passes)
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+__device__ __forceinline__ void st_cluster(float *p, uint32_t rank, float v) {      // *p of block `rank` of this cluster
+    uint32_t at = (uint32_t)__cvta_generic_to_shared(p), there;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(there) : "r"(at), "r"(rank));
+    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(there), "f"(v) : "memory");
+}
 template <typename WT, int DCH>
-__global__ void __launch_bounds__(delta_step_threads(DCH)) k_delta_step(const DeltaStepArgs a) {
+__global__ void __launch_bounds__(kDeltaThreads) k_delta_step(const DeltaStepArgs a) {
     pdl_launch_next();
+    cluster_arrive();                          // waited for before the first access to another block's shared memory
     constexpr uint32_t DP = DCH * 32u;
     extern __shared__ __align__(16) float sm[];
-    __shared__ float kq_s[kGemvMaxM], beta_s[kGemvMaxM];
-    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, sub = lane & 7u, nw = blockDim.x >> 5, h = blockIdx.x, D = a.D, VD = a.VD, T = a.T;
+    __shared__ float kq_s[kGemvMaxM], beta_s[kGemvMaxM], ss_s[kGemvMaxM][kDeltaBlocks];
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, sub = lane & 7u, nw = blockDim.x >> 5, h = blockIdx.y, D = a.D, VD = a.VD, T = a.T;
+    const uint32_t CB = delta_step_cols(VD), col_lo = min(VD, blockIdx.x * CB), nc = min(VD, col_lo + CB) - col_lo;      // this block's value columns
     const WT *a2 = static_cast<const WT *>(a.a2), *g2 = static_cast<const WT *>(a.g2);
-    if (a2) prefetch_weight_rows(a2 + (size_t)h * D * a.ra, sizeof(WT), a.ra, a.ra, D, warp, nw, 8u);
-    if (g2) prefetch_weight_rows(g2 + (size_t)h * VD * a.rg, sizeof(WT), a.rg, a.rg, VD, warp, nw, 8u);
+    if (a2) prefetch_weight_rows(a2 + (size_t)h * D * a.ra, sizeof(WT), a.ra, a.ra, D, warp, nw, 16u);
+    if (g2) prefetch_weight_rows(g2 + ((size_t)h * VD + col_lo) * a.rg, sizeof(WT), a.rg, a.rg, nc, warp, nw, 4u);
     pdl_wait();
-    float *q_s = sm, *k_s = q_s + kGemvMaxM * DP, *g_s = k_s + kGemvMaxM * DP, *o_s = g_s + kGemvMaxM * DP, *gate_s = o_s + kGemvMaxM * VD;
+    float *q_s = sm, *k_s = q_s + kGemvMaxM * DP, *g_s = k_s + kGemvMaxM * DP, *o_s = g_s + kGemvMaxM * DP, *gate_s = o_s + kGemvMaxM * CB;
     const uint32_t GD = a.G * D, C = 2u * GD + a.H * VD, gk = (h / (a.H / a.G)) * D, groups = blockDim.x >> 3;
     const bool dvec = (D & 3u) == 0;
-    float S[DCH][4];
-    auto load_state = [&](uint32_t col) {
-        const float *Sp = a.S + ((size_t)h * VD + col) * D;
+    float S[DCH][4], v_r[kGemvMaxM];
+    // a column's state and its values of every token; j: column of this block
+    auto load_column = [&](uint32_t j) {
+        const float *Sp = a.S + ((size_t)h * VD + col_lo + j) * D;
 #pragma unroll
         for (int c = 0; c < DCH; c++) {
             const uint32_t d = (sub + 8u * c) * 4u;
 #pragma unroll
             for (int e = 0; e < 4; e++) S[c][e] = 0.0f;
-            if (col < VD && d < D) {
+            if (j < nc && d < D) {
                 if (dvec) { const float4 v = *reinterpret_cast<const float4 *>(Sp + d); S[c][0] = v.x; S[c][1] = v.y; S[c][2] = v.z; S[c][3] = v.w; }
                 else {
 #pragma unroll
@@ -810,48 +885,51 @@ __global__ void __launch_bounds__(delta_step_threads(DCH)) k_delta_step(const De
                 }
             }
         }
+#pragma unroll
+        for (uint32_t t = 0; t < kGemvMaxM; t++) v_r[t] = (t < T && j < nc) ? a.cv[(size_t)t * C + 2u * GD + h * VD + col_lo + j] : 0.0f;
     };
-    load_state(tid >> 3);                      // in flight while the vectors are made
+    load_column(tid >> 3);                     // in flight while the vectors are made
+    const float rate = a.rate[h];
     for (uint32_t t = warp; t < T; t += nw) {  // unit vectors of a token
         const float *q = a.cv + (size_t)t * C + gk, *k = q + GD;
-        float sq = 0.0f, sk = 0.0f, sx = 0.0f;
-        for (uint32_t d = lane; d < DP; d += 32u) {
-            const float qv = d < D ? q[d] : 0.0f, kv = d < D ? k[d] : 0.0f;
-            q_s[t * DP + d] = qv; k_s[t * DP + d] = kv;
-            sq = fmaf(qv, qv, sq); sk = fmaf(kv, kv, sk); sx = fmaf(qv, kv, sx);
-        }
-        const float rq = a.qscale / sqrtf(warp_sum(sq) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(sk) + 1e-6f);
-        sx = warp_sum(sx);
-        float gh = 1.0f;
-        if (!a2) gh = delta_decay(a.rate[h], softplusf_(a.p[(size_t)t * a.ld + a.a0 + h] + a.dt_bias[h]));
-        for (uint32_t d = lane; d < DP; d += 32u) { q_s[t * DP + d] *= rq; k_s[t * DP + d] *= rk; if (!a2) g_s[t * DP + d] = gh; }
-        if (lane == 0) { kq_s[t] = sx * rq * rk; beta_s[t] = sigmoidf_(a.p[(size_t)t * a.ld + a.b0 + h]); }
+        float qr[DCH], kr[DCH], sq = 0.0f, sk = 0.0f, sx = 0.0f;
+        const float braw = a.p[(size_t)t * a.ld + a.b0 + h], araw = a2 ? 0.0f : a.p[(size_t)t * a.ld + a.a0 + h] + a.dt_bias[h];
+#pragma unroll
+        for (int c = 0; c < DCH; c++) { const uint32_t d = lane + 32u * c; qr[c] = d < D ? q[d] : 0.0f; kr[c] = d < D ? k[d] : 0.0f; }
+#pragma unroll
+        for (int c = 0; c < DCH; c++) { sq = fmaf(qr[c], qr[c], sq); sk = fmaf(kr[c], kr[c], sk); sx = fmaf(qr[c], kr[c], sx); }
+        sq = warp_sum(sq); sk = warp_sum(sk); sx = warp_sum(sx);
+        const float rq = a.qscale / sqrtf(sq + 1e-6f), rk = 1.0f / sqrtf(sk + 1e-6f), gh = a2 ? 1.0f : delta_decay(rate, softplusf_(araw));
+#pragma unroll
+        for (int c = 0; c < DCH; c++) { const uint32_t d = t * DP + lane + 32u * c; q_s[d] = qr[c] * rq; k_s[d] = kr[c] * rk; if (!a2) g_s[d] = gh; }
+        if (lane == 0) { kq_s[t] = sx * rq * rk; beta_s[t] = sigmoidf_(braw); }
     }
     if (a2) {
         const bool vec = a.ra % WVec<WT>::N == 0 && ((a.a0 | a.ld) & 3u) == 0 && (reinterpret_cast<uintptr_t>(a2) & 15u) == 0;
-        const float rate = a.rate[h];
         for (uint32_t r0 = 0; r0 < DP; r0 += groups) {      // a warp's lanes stay together: the row sums are shuffles
-            const uint32_t r = r0 + (tid >> 3);
+            const uint32_t r = r0 + (tid >> 3), rr = h * D + min(r, D - 1u);
+            const float bias = a.dt_bias[rr];
             float z[kGemvMaxM];
-            lane8_dots<WT>(a2 + (size_t)(h * D + min(r, D - 1u)) * a.ra, a.p + a.a0, a.ld, T, a.ra, vec, a.round_a != 0, sub, z);
-            if (sub < T && r < DP) g_s[sub * DP + r] = r < D ? delta_decay(rate, softplusf_(pick_row(z, (int32_t)sub) + a.dt_bias[h * D + r])) : 1.0f;
+            lane8_dots<WT>(a2 + (size_t)rr * a.ra, a.p + a.a0, a.ld, T, a.ra, vec, a.round_a != 0, sub, z);
+            if (sub < T && r < DP) g_s[sub * DP + r] = r < D ? delta_decay(rate, softplusf_(pick_row(z, (int32_t)sub) + bias)) : 1.0f;
         }
     }
     if (g2) {
         const bool vec = a.rg % WVec<WT>::N == 0 && ((a.g0 | a.ld) & 3u) == 0 && (reinterpret_cast<uintptr_t>(g2) & 15u) == 0;
-        for (uint32_t r0 = 0; r0 < VD; r0 += groups) {
+        for (uint32_t r0 = 0; r0 < nc; r0 += groups) {
             const uint32_t r = r0 + (tid >> 3);
             float z[kGemvMaxM];
-            lane8_dots<WT>(g2 + (size_t)(h * VD + min(r, VD - 1u)) * a.rg, a.p + a.g0, a.ld, T, a.rg, vec, a.round_a != 0, sub, z);
-            if (sub < T && r < VD) gate_s[sub * VD + r] = sigmoidf_(pick_row(z, (int32_t)sub));
+            lane8_dots<WT>(g2 + ((size_t)h * VD + col_lo + min(r, nc - 1u)) * a.rg, a.p + a.g0, a.ld, T, a.rg, vec, a.round_a != 0, sub, z);
+            if (sub < T && r < nc) gate_s[sub * CB + r] = sigmoidf_(pick_row(z, (int32_t)sub)) * a.gain[col_lo + r];
         }
-    } else for (uint32_t i = tid; i < T * VD; i += blockDim.x) gate_s[i] = siluf_(a.p[(size_t)(i / VD) * a.ld + a.g0 + h * VD + i % VD]);
+    } else for (uint32_t i = tid; i < T * nc; i += blockDim.x) gate_s[(i / nc) * CB + i % nc] = siluf_(a.p[(size_t)(i / nc) * a.ld + a.g0 + h * VD + col_lo + i % nc]) * a.gain[col_lo + i % nc];
     __syncthreads();
-    for (uint32_t c0 = 0; c0 < VD; c0 += groups) {
-        const uint32_t col = c0 + (tid >> 3);
-        if (c0) load_state(col);
-        for (uint32_t t = 0; t < T; t++) {
-            const float v = col < VD ? a.cv[(size_t)t * C + 2u * GD + h * VD + col] : 0.0f;
+    for (uint32_t c0 = 0; c0 < nc; c0 += groups) {
+        const uint32_t j = c0 + (tid >> 3);
+        if (c0) load_column(j);
+#pragma unroll
+        for (uint32_t t = 0; t < kGemvMaxM; t++) {
+            if (t >= T) break;
             float pk = 0.0f, pq = 0.0f;
 #pragma unroll
             for (int c = 0; c < DCH; c++) {
@@ -863,16 +941,16 @@ __global__ void __launch_bounds__(delta_step_threads(DCH)) k_delta_step(const De
             }
 #pragma unroll
             for (int off = 4; off > 0; off >>= 1) { pk += __shfl_xor_sync(0xffffffffu, pk, off); pq += __shfl_xor_sync(0xffffffffu, pq, off); }
-            const float u = beta_s[t] * (v - pk);
-            if (sub == 0 && col < VD) o_s[t * VD + col] = fmaf(kq_s[t], u, pq);
+            const float u = beta_s[t] * (v_r[t] - pk);
+            if (sub == 0 && j < nc) o_s[t * CB + j] = fmaf(kq_s[t], u, pq);
 #pragma unroll
             for (int c = 0; c < DCH; c++) {
                 const float4 kv = *reinterpret_cast<const float4 *>(k_s + t * DP + (sub + 8u * c) * 4u);
                 S[c][0] = fmaf(kv.x, u, S[c][0]); S[c][1] = fmaf(kv.y, u, S[c][1]); S[c][2] = fmaf(kv.z, u, S[c][2]); S[c][3] = fmaf(kv.w, u, S[c][3]);
             }
         }
-        if (col < VD) {
-            float *Sp = a.S + ((size_t)h * VD + col) * D;
+        if (j < nc) {
+            float *Sp = a.S + ((size_t)h * VD + col_lo + j) * D;
 #pragma unroll
             for (int c = 0; c < DCH; c++) {
                 const uint32_t d = (sub + 8u * c) * 4u;
@@ -886,11 +964,21 @@ __global__ void __launch_bounds__(delta_step_threads(DCH)) k_delta_step(const De
         }
     }
     __syncthreads();
-    for (uint32_t t = warp; t < T; t += nw) {
+    cluster_wait();                            // every block of the cluster runs
+    for (uint32_t t = warp; t < T; t += nw) {  // this block's share of the head's sum of squares, to every block of the head
         float s = 0.0f;
-        for (uint32_t j = lane; j < VD; j += 32u) s = fmaf(o_s[t * VD + j], o_s[t * VD + j], s);
-        const float rinv = 1.0f / sqrtf(warp_sum(s) / (float)VD + a.eps);
-        for (uint32_t j = lane; j < VD; j += 32u) a.out[((size_t)t * a.H + h) * VD + j] = o_s[t * VD + j] * rinv * a.gain[j] * gate_s[t * VD + j];
+        for (uint32_t j = lane; j < nc; j += 32u) s = fmaf(o_s[t * CB + j], o_s[t * CB + j], s);
+        s = warp_sum(s);
+        if (lane < gridDim.x) st_cluster(&ss_s[t][blockIdx.x], lane, s);
+    }
+    __syncwarp();
+    cluster_arrive();
+    cluster_wait();
+    for (uint32_t i = tid; i < T * nc; i += blockDim.x) {
+        const uint32_t t = i / nc, j = i % nc;
+        float s = 0.0f;
+        for (uint32_t r = 0; r < gridDim.x; r++) s += ss_s[t][r];
+        a.out[((size_t)t * a.H + h) * VD + col_lo + j] = o_s[t * CB + j] / sqrtf(s / (float)VD + a.eps) * gate_s[t * CB + j];
     }
 }
 
