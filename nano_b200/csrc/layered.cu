@@ -182,7 +182,7 @@ struct LayeredEngine : nb::EngineBase {
     // short portions of a Dynamic-Tanh design: the residual update that follows a sublayer rides on the sublayer's last product
     struct ResEpi { bool on = false; Dyt post{}, pre{}; float *out = nullptr, *keep = nullptr; } res;
     float *b_dpart = nullptr, *b_sseg = nullptr, *b_sdx = nullptr, *b_sdy = nullptr, *b_f2 = nullptr, *b_hg = nullptr, *b_sh2 = nullptr, *b_sg = nullptr, *b_wrow = nullptr; uint32_t *b_dtick = nullptr;
-    // gated delta rule: convolved channels of a short portion; what the preparation hands the scan; low-rank products; outputs before and after the gate
+    // gated delta rule: convolved channels of a short portion; what the preparation hands the scan (chunk blocks, values); low-rank products; outputs before and after the gate
     float *b_gcv = nullptr, *b_gblk = nullptr, *b_gv = nullptr, *b_gsp = nullptr, *b_gt = nullptr, *b_go = nullptr, *b_ga = nullptr;
     float *b_gpart = nullptr; uint32_t *b_gtick = nullptr;      // grouped-query attention: partials and tickets of the key splits
     uint32_t *ids_dev = nullptr, *want_dev = nullptr, *next_dev = nullptr, *tok_host = nullptr; uint8_t *seen = nullptr;

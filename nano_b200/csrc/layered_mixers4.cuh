@@ -10,9 +10,9 @@
 //                        k_gqa_decode (the same for short portions: norm, rotation, cache write, scores, softmax and merge of the key
 //                        splits in one launch)
 //   gated delta rule     per head  S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q,  g one number or one per key channel.
-//                        k_delta_prep (convolution, silu, unit vectors, step size, decay, and the products between tokens that let
-//                        kDeltaChunk tokens be solved together), k_delta_scan (the recurrence of a long portion, kDeltaChunk tokens per
-//                        step), k_delta_step (short portions: everything after the convolution up to the gated, normed output)
+//                        k_delta_prep (convolution, silu, unit vectors, step size, decay, and everything that lets kDeltaChunk tokens be
+//                        solved together), k_delta_scan (the recurrence of a long portion, kDeltaChunk tokens per step), k_delta_step
+//                        (short portions: everything after the convolution up to the gated, normed output, a cluster of blocks per head)
 #pragma once
 #include "layered_mixers3.cuh"
 
