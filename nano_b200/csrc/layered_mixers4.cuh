@@ -801,8 +801,8 @@ __global__ void __launch_bounds__(256, 2) k_delta_scan(const DeltaScanArgs a) {
 }
 
 // Short portions (T <= kGemvMaxM): a cluster of blocks per head, each with a share of its value columns, from the convolved channels (an
-// epilogue of the joint product) to the normed and gated output; the blocks exchange their columns' sums of squares through each other's
-// shared memory.  8 lanes share a value column.  Low-rank decay and gate: their second products, W_a2 (a1) and W_g2 (g1) with a1, g1
+// epilogue of the joint product) to the normed and gated output; the blocks exchange their parts of the decays and their columns' sums of
+// squares through each other's shared memory.  8 lanes share a value column.  Low-rank decay and gate: their second products, W_a2 (a1) and W_g2 (g1) with a1, g1
 // columns of the joint product, are made here for the head's own rows (round_a: the operand rounded to bf16 first, as a tensor-core
 // product would).  Without them the decay is one number per head (column a0 + h) and the gate silu of H VD columns at g0.
 constexpr uint32_t kDeltaBlocks = 4;       // blocks per head at most
@@ -862,7 +862,8 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_step(const DeltaStepArg
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, sub = lane & 7u, nw = blockDim.x >> 5, h = blockIdx.y, D = a.D, VD = a.VD, T = a.T;
     const uint32_t CB = delta_step_cols(VD), col_lo = min(VD, blockIdx.x * CB), nc = min(VD, col_lo + CB) - col_lo;      // this block's value columns
     const WT *a2 = static_cast<const WT *>(a.a2), *g2 = static_cast<const WT *>(a.g2);
-    if (a2) prefetch_weight_rows(a2 + (size_t)h * D * a.ra, sizeof(WT), a.ra, a.ra, D, warp, nw, 16u);
+    const uint32_t part = DP / gridDim.x, lo = blockIdx.x * part, hi = lo + part;      // this block's share of the head's decays
+    if (a2 && lo < D) prefetch_weight_rows(a2 + ((size_t)h * D + lo) * a.ra, sizeof(WT), a.ra, a.ra, min(hi, D) - lo, warp, nw, 8u);
     if (g2) prefetch_weight_rows(g2 + ((size_t)h * VD + col_lo) * a.rg, sizeof(WT), a.rg, a.rg, nc, warp, nw, 4u);
     pdl_wait();
     float *q_s = sm, *k_s = q_s + kGemvMaxM * DP, *g_s = k_s + kGemvMaxM * DP, *o_s = g_s + kGemvMaxM * DP, *gate_s = o_s + kGemvMaxM * CB;
@@ -906,12 +907,18 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_step(const DeltaStepArg
     }
     if (a2) {
         const bool vec = a.ra % WVec<WT>::N == 0 && ((a.a0 | a.ld) & 3u) == 0 && (reinterpret_cast<uintptr_t>(a2) & 15u) == 0;
-        for (uint32_t r0 = 0; r0 < DP; r0 += groups) {      // a warp's lanes stay together: the row sums are shuffles
+        // the head's decays are shared work: every block makes its part of the rows and hands them to all blocks of the head
+        __syncwarp();
+        cluster_wait();                        // every block of the cluster runs
+        for (uint32_t r0 = lo; r0 < hi; r0 += groups) {      // a warp's lanes stay together: the row sums are shuffles
             const uint32_t r = r0 + (tid >> 3), rr = h * D + min(r, D - 1u);
             const float bias = a.dt_bias[rr];
             float z[kGemvMaxM];
             lane8_dots<WT>(a2 + (size_t)rr * a.ra, a.p + a.a0, a.ld, T, a.ra, vec, a.round_a != 0, sub, z);
-            if (sub < T && r < DP) g_s[sub * DP + r] = r < D ? delta_decay(rate, softplusf_(pick_row(z, (int32_t)sub) + bias)) : 1.0f;
+            if (sub < T && r < hi) {
+                const float gv = r < D ? delta_decay(rate, softplusf_(pick_row(z, (int32_t)sub) + bias)) : 1.0f;
+                for (uint32_t b = 0; b < gridDim.x; b++) st_cluster(&g_s[sub * DP + r], b, gv);
+            }
         }
     }
     if (g2) {
@@ -923,7 +930,8 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_step(const DeltaStepArg
             if (sub < T && r < nc) gate_s[sub * CB + r] = sigmoidf_(pick_row(z, (int32_t)sub)) * a.gain[col_lo + r];
         }
     } else for (uint32_t i = tid; i < T * nc; i += blockDim.x) gate_s[(i / nc) * CB + i % nc] = siluf_(a.p[(size_t)(i / nc) * a.ld + a.g0 + h * VD + col_lo + i % nc]) * a.gain[col_lo + i % nc];
-    __syncthreads();
+    __syncwarp();
+    if (a2) { cluster_arrive(); cluster_wait(); } else __syncthreads();
     for (uint32_t c0 = 0; c0 < nc; c0 += groups) {
         const uint32_t j = c0 + (tid >> 3);
         if (c0) load_column(j);
@@ -964,7 +972,7 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_step(const DeltaStepArg
         }
     }
     __syncthreads();
-    cluster_wait();                            // every block of the cluster runs
+    if (!a2) cluster_wait();                   // every block of the cluster runs
     for (uint32_t t = warp; t < T; t += nw) {  // this block's share of the head's sum of squares, to every block of the head
         float s = 0.0f;
         for (uint32_t j = lane; j < nc; j += 32u) s = fmaf(o_s[t * CB + j], o_s[t * CB + j], s);
