@@ -128,19 +128,23 @@ __global__ void __launch_bounds__(256) k_qk_norm_rope(const GqaArgs a) {
         if (a.wk) rk = 1.0f / sqrtf(s.y / (float)KW + a.eps);
     }
     const float2 *cs = a.tab + (size_t)pos * half;
-    // q in place: a thread owns both coordinates of a pair
-    const uint32_t per = a.D - half;
-    for (uint32_t i = threadIdx.x; i < a.H * per; i += blockDim.x) {
-        const uint32_t h = i / per, e = i % per;
-        float *qh = q + h * a.D;
-        const float *w = a.wq ? a.wq + h * a.D : nullptr;
-        if (e < half) {
-            const float u = rot_half_at(qh, w, rq, e, half, cs) * a.scale, z = rot_half_at(qh, w, rq, e + half, half, cs) * a.scale;
-            qh[e] = u; qh[e + half] = z;
-        } else qh[e + half] = rot_half_at(qh, w, rq, e + half, half, cs) * a.scale;
-    }
+    // a warp per head; q in place (a lane owns both coordinates of a pair), k into the token's cache row, v beside it
+    const uint32_t per = a.D - half, warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, nw = blockDim.x >> 5;
     float *row = a.cache + ((size_t)a.table[pos / kPage] * kPage + pos % kPage) * a.RL;
-    for (uint32_t i = threadIdx.x; i < KW; i += blockDim.x) row[i] = rot_half_at(k + (i / a.D) * a.D, a.wk ? a.wk + (i / a.D) * a.D : nullptr, rk, i % a.D, half, cs);
+    for (uint32_t h = warp; h < a.H + a.G; h += nw) {
+        const bool isq = h < a.H;
+        const uint32_t hh = (isq ? h : h - a.H) * a.D;
+        const float *src = (isq ? q : k) + hh, *w = isq ? (a.wq ? a.wq + hh : nullptr) : (a.wk ? a.wk + hh : nullptr);
+        float *dst = isq ? q + hh : row + hh;
+        const float r = isq ? rq * a.scale : rk;
+        for (uint32_t e = lane; e < per; e += 32u) {
+            if (e < half) {
+                const float u = src[e] * r * (w ? w[e] : 1.0f), z = src[e + half] * r * (w ? w[e + half] : 1.0f);
+                const float2 c = cs[e];
+                dst[e] = u * c.x - z * c.y; dst[e + half] = z * c.x + u * c.y;
+            } else dst[e + half] = src[e + half] * r * (w ? w[e + half] : 1.0f);
+        }
+    }
     for (uint32_t i = threadIdx.x; i < a.RL - KW; i += blockDim.x) row[KW + i] = i < a.G * a.VD ? v[i] : 0.0f;
 }
 
