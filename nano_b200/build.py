@@ -39,7 +39,7 @@ def _newer(target: str, sources) -> bool:
 UNITS = {
     "api.cu": ["family.h", "modeldir.h", "../../include/nano_b200.h"],
     "modeldir.cu": ["modeldir.h"],
-    "layered.cu": ["layered_kernels.cuh", "layered_mixers.cuh", "layered_mixers2.cuh", "layered_mixers3.cuh", "layered_mixers4.cuh", "family.h", "modeldir.h", "sample_host.h", "../../include/nano_b200.h"],
+    "layered.cu": ["layered_kernels.cuh", "layered_mixers.cuh", "layered_mixers2.cuh", "layered_mixers3.cuh", "layered_mixers4.cuh", "layered_mixers5.cuh", "family.h", "modeldir.h", "sample_host.h", "../../include/nano_b200.h"],
     "engine.cu": ["kernels.cuh", "expf_ref.cuh", "stream_args.h", "stream_host.h", "sample_host.h", "family.h", "../../include/nano_b200.h"],
     "stream.cu": ["kernels.cuh", "expf_ref.cuh", "stream_args.h", "stream_host.h", "stream.cuh"],
     "sample.cu": ["kernels.cuh", "expf_ref.cuh", "sample_host.h"],
@@ -57,7 +57,8 @@ def build_engine(force: bool = False, verbose: bool = False, units=None, target:
     units / target: a library of a subset of the families (build_layered)."""
     os.makedirs(LIB, exist_ok=True)
     target = target or ENGINE_SO
-    base = [NVCC, "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC"]
+    base = [NVCC, "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC",
+            "--split-compile", "0"]          # the kernels of one unit are optimised side by side
     if verbose:
         base.insert(1, "-Xptxas=-v")
     objs, procs = [], []

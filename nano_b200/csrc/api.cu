@@ -43,6 +43,7 @@ const DirFamily kDirFamilies[] = {
     {"Gokinex", nb_family_layered_create, "layered.cu"},
     {"Vumunex", nb_family_layered_create, "layered.cu"},
     {"Kadesun", nb_family_layered_create, "layered.cu"},
+    {"Fidatar", nb_family_layered_create, "layered.cu"},
 };
 }  // namespace
 

@@ -25,6 +25,11 @@
 // "parallel" (a grouped-query attention with query/key norm over the whole projection, rotary positions on half pairs, soft-capped
 // scores, a sink and one sigmoid gate per head, side by side with a gated delta rule whose decay is one number per key channel and whose
 // decay and output gate are low-rank products; each branch normed, then averaged); feed-forward "dense" (gated silu), or none.
+// "Fidatar" -- sequential sublayers that read the residual itself, which is normed after every sum, x <- rms_norm(alpha x + sublayer(x)) w;
+// the token row times a fixed scale; mixers "attention" (grouped-query attention inside fixed blocks of positions, with biases, query/key
+// norm per head, rescaled rotary positions on half pairs and one added to the softmax denominator) and "mlstm" (a matrix memory per head
+// with exponential input and forget gates); feed-forward "dense" (squared relu) or "moe" (squared-relu experts chosen by sigmoid scores
+// inside the best groups of experts), or none; soft-capped logits.
 // "Famudra" -- parallel layers  x <- x + (mixer(shift(norm1 x)) + ff(norm2 x))  with scalar-gain RMS norms and a
 // token shift on the mixer input; mixers "rglru" (gelu branch x conv + real-gated linear recurrent unit) and "latent_attention"
 // (queries and keys/values through normed low-rank latents, no positions, causal softmax); feed-forward "moe" (top-k routed
@@ -60,6 +65,7 @@
 #include "layered_mixers2.cuh"
 #include "layered_mixers3.cuh"
 #include "layered_mixers4.cuh"
+#include "layered_mixers5.cuh"
 #include "modeldir.h"
 #include "sample_host.h"
 
@@ -72,13 +78,14 @@ namespace {
 
 struct Weight { void *p = nullptr; uint32_t rows = 0, cols = 0; };
 
-enum MixerType { MIX_RGLRU = 0, MIX_LATENT_ATTN = 1, MIX_RETENTION = 2, MIX_WINDOW_SSM = 3, MIX_DIFF_ATTN = 4, MIX_SSD = 5, MIX_DELTA = 6, MIX_ATTN_DELTA = 7 };
+enum MixerType { MIX_RGLRU = 0, MIX_LATENT_ATTN = 1, MIX_RETENTION = 2, MIX_WINDOW_SSM = 3, MIX_DIFF_ATTN = 4, MIX_SSD = 5, MIX_DELTA = 6, MIX_ATTN_DELTA = 7, MIX_GQA = 8, MIX_MEMORY = 9 };
 // how a layer combines its sublayers: Famudra's parallel form with a token shift and scalar-gain norms, or sequential sublayers
 // between an input norm and an output norm each (vector gains stored around zero)
 // or pre-norm sublayers over hyper-connected residual streams (bias-free layer norms)
 // or sequential sublayers that read the residual itself and pass a norm on the way out (plain vector gains)
-enum LayerForm { FORM_PARALLEL_SHIFT = 0, FORM_SANDWICH = 1, FORM_HYPER = 2, FORM_POST = 3 };
-enum FfKind { FF_NONE = 0, FF_MOE = 1, FF_DENSE_POLY = 2, FF_DENSE_GLU = 3, FF_MOE_SCORED = 4, FF_DENSE_GELU = 5 };
+// or sequential sublayers that read the residual itself, with a norm of the sum (plain vector gains)
+enum LayerForm { FORM_PARALLEL_SHIFT = 0, FORM_SANDWICH = 1, FORM_HYPER = 2, FORM_POST = 3, FORM_POST_LN = 4 };
+enum FfKind { FF_NONE = 0, FF_MOE = 1, FF_DENSE_POLY = 2, FF_DENSE_GLU = 3, FF_MOE_SCORED = 4, FF_DENSE_GELU = 5, FF_DENSE_RELU2 = 6 };
 // the norms of the sequential form: unit RMS times a vector gain stored around zero, or Dynamic Tanh
 enum NormKind { NORM_RMS_ZERO = 0, NORM_DYT = 1 };
 
@@ -120,7 +127,7 @@ struct Layer {
     // state-space duality: proj = [z | x | B | C | dt]; H heads of vdim, mN states, G groups, m_taps, m_conv, m_conv_b, dt_b, A = exp(A_log)
     // per head, Dv per head; the output is normed in `parts` equal parts with the gain gn
     uint32_t parts = 0; float *gn = nullptr;
-    // output-normed form: gains after the mixer and after the feed-forward
+    // output-normed form and the form with norms of the sum: gains after the mixer and after the feed-forward
     float *pn1 = nullptr, *pn2 = nullptr;
     // gated delta rule (MIX_DELTA, and one branch of MIX_ATTN_DELTA): dH heads of value size dVD over dG query/key heads of dD; columns of the
     // joint product: convolved channels [q | k | v] from c_conv, step size c_b, decay c_a (a1 of rank ra, or one number per head), gate c_g
@@ -129,18 +136,22 @@ struct Layer {
     uint32_t dH = 0, dG = 0, dD = 0, dVD = 0, d_taps = 0, ra = 0, rg = 0, c_conv = 0, c_b = 0, c_a = 0, c_g = 0, c_hg = 0, a_half = 0;
     float *d_conv = nullptr, *d_bias = nullptr, *d_rate = nullptr, *d_gain = nullptr, *qn = nullptr, *kn = nullptr, *out1 = nullptr, *out2 = nullptr, mix_w = 1.0f;
     Weight a2, g2, d_o;
+    // grouped-query attention (MIX_GQA, and one branch of MIX_ATTN_DELTA): block_size (0: causal), norms per head or over the projection
+    uint32_t block_size = 0; bool head_norm = false;
+    // matrix memory: proj = [q | k | v | g | i | f] (biases in proj_b), H heads of dim and vdim, gain gn of all heads' values
+    float gate_cap = 0.0f; uint32_t c_if = 0;
     // feed-forward
     int ff_kind = FF_NONE; float *act = nullptr;
     bool has_mlp = false, has_shared = false;
     // scored experts: how the router weighs (k_route's mode), whether the weight scales what the expert reads (else its output), whether
     // the shared expert sits behind a gate row of the router, the gated unit (k_gemv's glu) and its limits
     uint32_t route_mode = 1, glu_kind = 2; bool score_in = true, sh_gate = false; float limit = 0.0f, slimit = 0.0f;
-    uint32_t NE = 0, top = 0, ff = 0, sff = 0;
+    uint32_t NE = 0, top = 0, ff = 0, sff = 0, groups = 1, keep_groups = 1; float route_scale = 1.0f;      // groups: neighbouring experts of which only the best can be chosen (k_route's mode 3)
     float *router = nullptr;
     Weight up, down, sup, sdown;
 };
 
-struct Run { uint32_t layer = 0; bool add_embed = false; size_t st_prev = 0, st_S = 0, st_conv = 0, st_conv2 = 0; float *cache = nullptr; };
+struct Run { uint32_t layer = 0; bool add_embed = false; size_t st_prev = 0, st_S = 0, st_conv = 0, st_conv2 = 0, st_n = 0, st_m = 0; float *cache = nullptr; };
 
 struct Seq { bool live = false; uint32_t len = 0; std::vector<uint32_t> pages; };
 
@@ -184,9 +195,12 @@ struct LayeredEngine : nb::EngineBase {
     float *b_dpart = nullptr, *b_sseg = nullptr, *b_sdx = nullptr, *b_sdy = nullptr, *b_f2 = nullptr, *b_hg = nullptr, *b_sh2 = nullptr, *b_sg = nullptr, *b_wrow = nullptr; uint32_t *b_dtick = nullptr;
     // gated delta rule: convolved channels of a short portion; what the preparation hands the scan (chunk blocks, values); low-rank products; outputs before and after the gate
     float *b_gcv = nullptr, *b_gblk = nullptr, *b_gv = nullptr, *b_gsp = nullptr, *b_gt = nullptr, *b_go = nullptr, *b_ga = nullptr;
+    // matrix memory: per head and token the gates' sums, per chunk the state before it
+    double *b_mfa = nullptr, *b_mfb = nullptr, *b_mfc = nullptr; float *b_mmt = nullptr, *b_mme = nullptr, *b_mS = nullptr, *b_mn = nullptr, *b_mo = nullptr;
     float *b_gpart = nullptr; uint32_t *b_gtick = nullptr;      // grouped-query attention: partials and tickets of the key splits
     uint32_t *ids_dev = nullptr, *want_dev = nullptr, *next_dev = nullptr, *tok_host = nullptr; uint8_t *seen = nullptr;
     uint32_t last_T = 0;
+    float alpha = 1.0f, logit_cap = 0.0f;      // norms of the sum: the residual's factor; soft cap of the logits (0: none)
     uint32_t S = 1; float res_mult = 1.0f; float *xs = nullptr;      // hyper-connected form: streams, the model's residual multiplier, the streams [S][chunk][E]
     uint32_t *dpos = nullptr, *zero_dev = nullptr;            // device-side position of a captured decode step; a constant 0
     bool branch_streams = true;      // a layer's feed-forward and shared expert on streams of their own (NB200_NO_BRANCH_STREAMS=1: one stream)
@@ -331,13 +345,23 @@ int load_latent_attn(Loader &ld, const nb::Json *m, const std::string &p, Layer 
     return ld.put_w(t, (uint32_t)(H * R), (uint32_t)D, &L->ukT);
 }
 
-int load_moe(Loader &ld, const nb::Json *f, const std::string &p, Layer *L, uint32_t E) {
+// squared-relu experts without biases.  sigmoid_groups: chosen by sigmoid scores inside the best groups (k_route's mode 3), else by a
+// softmax over the chosen
+int load_moe(Loader &ld, const nb::Json *f, const std::string &p, Layer *L, uint32_t E, bool sigmoid_groups = false) {
     const nb::Json *kind = f->get("kind");
     if (!kind || kind->t != nb::Json::Str || kind->str != "moe") return fail(NB200_EINVAL, "%s: feed-forward kind \"%s\" is not known", p.c_str(), kind && kind->t == nb::Json::Str ? kind->str.c_str() : "?");
     if (!u32_of(f->get("router"), "experts", &L->NE) || !u32_of(f->get("router"), "top", &L->top) || !u32_of(f->get("expert"), "ff", &L->ff))
         return fail(NB200_EINVAL, "%s: a moe feed-forward needs router.experts, router.top and expert.ff", p.c_str());
     if (!L->NE || !L->top || L->top > L->NE || !L->ff) return fail(NB200_EINVAL, "%s: experts %u / top %u / ff %u unusable", p.c_str(), L->NE, L->top, L->ff);
-    L->has_mlp = true; L->ff_kind = FF_MOE;
+    L->has_mlp = true; L->ff_kind = FF_MOE; L->route_mode = 0;
+    if (sigmoid_groups) {
+        const nb::Json *ro = f->get("router"); double sc = 1.0;
+        if (ro->present("groups") && (!u32_of(ro->get("groups"), "count", &L->groups) || !u32_of(ro->get("groups"), "keep", &L->keep_groups))) return fail(NB200_EINVAL, "%s: router.groups needs count and keep", p.c_str());
+        if (ro->present("scale") && !ro->number("scale", &sc)) return fail(NB200_EINVAL, "%s: router.scale must be a number", p.c_str());
+        L->route_mode = 3; L->route_scale = (float)sc;
+        if (!L->groups || L->NE % L->groups || !L->keep_groups || L->keep_groups > L->groups || L->top > L->keep_groups * (L->NE / L->groups))
+            return fail(NB200_EINVAL, "%s: experts %u / groups %u / kept %u / top %u unusable", p.c_str(), L->NE, L->groups, L->keep_groups, L->top);
+    }
     int r;
     if ((r = ld.vec(p + "router", {L->NE, E}, &L->router))) return r;
     std::vector<std::string> ups, downs; std::vector<uint64_t> ur, dr;
@@ -472,27 +496,41 @@ int joined_vec(Loader &ld, const std::vector<std::string> &names, const std::vec
 
 // (cos, sin) of position x frequency for `positions` positions, built in double.  f_i = base^(-2i/dims), rescaled by wavelength
 // l = 2 pi / f when `scaling` {factor, low, high, original} is given: kept where l < original / high, divided by factor where
-// l > original / low, and between the two blended, (1 - s) f / factor + s f with s = (original / l - low) / (high - low).
+// l > original / low, and between the two blended, (1 - s) f / factor + s f with s = (original / l - low) / (high - low);
+// with {factor, fast, slow, original} (YaRN) blended by a ramp over the pairs, from the pair that turns `fast` times over the original
+// length (kept) to the one that turns `slow` times (divided by factor), and cos and sin times 0.1 ln(factor) + 1.
 int rope_table(Loader &ld, const nb::Json *rot, const std::string &p, uint32_t dims, uint32_t positions, float2 **out) {
     double base, factor = 1.0, low = 0.0, high = 0.0, original = 0.0;
     if (!rot->number("base", &base) || !(base > 0.0)) return fail(NB200_EINVAL, "%s: rot needs a base > 0", p.c_str());
     const nb::Json *sc = rot->present("scaling") ? rot->get("scaling") : nullptr;
-    if (sc && (!sc->number("factor", &factor) || !sc->number("low", &low) || !sc->number("high", &high) || !sc->number("original", &original) || !(factor > 0.0) || !(high > low) || !(original > 0.0)))
+    const bool yarn = sc && sc->present("fast");
+    double fast = 0.0, slow = 0.0, amp = 1.0, ramp_lo = 0.0, ramp_hi = 0.0;
+    if (yarn) {
+        if (!sc->number("factor", &factor) || !sc->number("original", &original) || !sc->number("fast", &fast) || !sc->number("slow", &slow) || !(factor > 0.0) || !(original > 0.0) || !(fast > 0.0) || !(slow > 0.0))
+            return fail(NB200_EINVAL, "%s: rot.scaling needs factor, original, fast and slow, all > 0", p.c_str());
+        auto place = [&](double turns) { return (double)dims * log(original / (6.283185307179586476925286766559 * turns)) / (2.0 * log(base)); };
+        ramp_lo = std::max(floor(place(fast)), 0.0); ramp_hi = std::min(ceil(place(slow)), (double)dims - 1.0);
+        amp = 0.1 * log(factor) + 1.0;
+    }
+    if (sc && !yarn && (!sc->number("factor", &factor) || !sc->number("low", &low) || !sc->number("high", &high) || !sc->number("original", &original) || !(factor > 0.0) || !(high > low) || !(original > 0.0)))
         return fail(NB200_EINVAL, "%s: rot.scaling needs factor > 0, low < high and original > 0", p.c_str());
-    char key[160];
-    snprintf(key, sizeof key, "%u/%.17g/%d/%.17g/%.17g/%.17g/%.17g", dims, base, sc ? 1 : 0, factor, low, high, original);
+    char key[256];
+    snprintf(key, sizeof key, "%u/%.17g/%d/%.17g/%.17g/%.17g/%.17g/%.17g/%.17g", dims, base, sc ? (yarn ? 2 : 1) : 0, factor, low, high, original, fast, slow);
     for (auto &kv : ld.e->rot_tabs) if (kv.first == key) { *out = kv.second; return 0; }
     const uint32_t half = dims / 2u;
     const double two_pi = 6.283185307179586476925286766559;
     std::vector<float> tab((size_t)positions * half * 2);
     for (uint32_t i = 0; i < half; i++) {
         double f = pow(base, -2.0 * (double)i / (double)dims);
-        if (sc) {
+        if (yarn) {
+            const double ramp = std::min(std::max(((double)i - ramp_lo) / std::max(ramp_hi - ramp_lo, 0.001), 0.0), 1.0);
+            f = f / factor * ramp + f * (1.0 - ramp);
+        } else if (sc) {
             const double wave = two_pi / f;
             if (wave > original / low) f = f / factor;
             else if (!(wave < original / high)) { const double sm = (original / wave - low) / (high - low); f = (1.0 - sm) * f / factor + sm * f; }
         }
-        for (uint32_t q = 0; q < positions; q++) { const double a = (double)q * f; tab[((size_t)q * half + i) * 2] = (float)cos(a); tab[((size_t)q * half + i) * 2 + 1] = (float)sin(a); }
+        for (uint32_t q = 0; q < positions; q++) { const double a = (double)q * f; tab[((size_t)q * half + i) * 2] = (float)(amp * cos(a)); tab[((size_t)q * half + i) * 2 + 1] = (float)(amp * sin(a)); }
     }
     float *t = nullptr; int r;
     if ((r = ld.put_f32(tab, &t))) return r;
@@ -647,10 +685,10 @@ int load_latent_attn_direct(Loader &ld, const nb::Json *m, const std::string &p,
     return ld.put_w(t, (uint32_t)(H * R), (uint32_t)D, &L->ukT);
 }
 
-// dense feed-forward down(gelu(up h)) with the exact (erf) gelu
-int load_dense_gelu(Loader &ld, const nb::Json *f, const std::string &p, Layer *L, uint32_t E) {
+// dense feed-forward down(act(up h)); kind FF_DENSE_GELU: the exact (erf) gelu, FF_DENSE_RELU2: squared relu
+int load_dense_act(Loader &ld, const nb::Json *f, const std::string &p, Layer *L, uint32_t E, int kind) {
     if (!u32_of(f, "ff", &L->ff) || !L->ff) return fail(NB200_EINVAL, "%s: a dense feed-forward needs ff", p.c_str());
-    L->has_mlp = true; L->ff_kind = FF_DENSE_GELU;
+    L->has_mlp = true; L->ff_kind = kind;
     int r;
     if ((r = ld.stacked({p + "up"}, {L->ff}, E, &L->up))) return r;
     return ld.stacked({p + "down"}, {E}, L->ff, &L->down);
@@ -719,27 +757,73 @@ int load_delta(Loader &ld, const nb::Json *m, const std::string &p, Layer *L, ui
 
 constexpr size_t kGqaSmemMax = 227 * 1024;
 inline int gqa_vj(uint32_t vdim) { return vdim <= 64 ? 1 : vdim <= 128 ? 2 : 4; }
+// sizes, scale, cap, positions and blocks of a grouped-query attention (p: what messages call it)
+int load_gqa_sizes(Loader &ld, const nb::Json *m, const std::string &p, Layer *L, uint32_t positions) {
+    double sc;
+    if (!u32_of(m, "heads", &L->H) || !u32_of(m, "kv_heads", &L->G) || !u32_of(m, "dim", &L->dim) || !u32_of(m, "vdim", &L->vdim) || !m->number("scale", &sc))
+        return fail(NB200_EINVAL, "%s: an attention needs heads, kv_heads, dim, vdim and scale", p.c_str());
+    L->scale = (float)sc;
+    if (!L->H || !L->G || L->H % L->G || !L->dim || !L->vdim) return fail(NB200_EINVAL, "%s: heads %u / kv_heads %u / dim %u / vdim %u unusable", p.c_str(), L->H, L->G, L->dim, L->vdim);
+    if (L->dim > 256 || L->vdim > 256) return fail(NB200_EINVAL, "%s: dim %u or vdim %u above 256 has no attention kernel", p.c_str(), L->dim, L->vdim);
+    if (m->present("softcap")) { double c; if (!m->number("softcap", &c) || !(c >= 0.0)) return fail(NB200_EINVAL, "%s: softcap must be a number >= 0", p.c_str()); L->softcap = (float)c; }
+    if (m->present("rot")) {
+        const nb::Json *rot = m->get("rot");
+        int r;
+        if (!u32_of(rot, "dims", &L->rot_dims) || L->rot_dims > L->dim || (L->rot_dims & 1u)) return fail(NB200_EINVAL, "%s: rot needs an even dims <= dim", p.c_str());
+        if (L->rot_dims && (r = rope_table(ld, rot, p, L->rot_dims, positions, &L->rot_tab))) return r;
+        L->a_half = L->rot_dims / 2u;
+    }
+    if (m->present("mask") && (!u32_of(m->get("mask"), "size", &L->block_size) || !L->block_size)) return fail(NB200_EINVAL, "%s: mask.size must be a positive integer", p.c_str());
+    L->RL = (L->G * (L->dim + L->vdim) + 3u) & ~3u;
+    return 0;
+}
+// a vector of J's columns: parts {column, tensor, length}, zeros elsewhere
+struct JointPart { uint32_t at; std::string name; uint64_t n; };
+int joint_bias(Loader &ld, const JointRows &J, const std::vector<JointPart> &parts, float **dst) {
+    std::vector<float> all(J.cols, 0.0f);
+    for (const JointPart &q : parts) {
+        std::vector<float> h; std::vector<uint64_t> sh; int r;
+        if ((r = ld.host_f32(q.name, &h, &sh)) || (r = ld.expect(q.name, sh, {q.n}))) return r;
+        std::copy(h.begin(), h.end(), all.begin() + q.at);
+    }
+    return ld.put_f32(all, dst);
+}
+// grouped-query attention alone: biases on q, k and v, norms per head with gains shared by the heads, blocks of positions, and a softmax
+// with one added to its denominator (a sink of score zero for every head)
+int load_gqa(Loader &ld, const nb::Json *m, const std::string &p, Layer *L, uint32_t E, uint32_t positions) {
+    JointRows J; int r;
+    if ((r = load_gqa_sizes(ld, m, p, L, positions))) return r;
+    const uint64_t H = L->H, G = L->G, D = L->dim, VD = L->vdim;
+    if ((r = J.add(ld, p + "q", H * D, E, nullptr)) || (r = J.add(ld, p + "k", G * D, E, nullptr)) || (r = J.add(ld, p + "v", G * VD, E, nullptr)) || (r = J.put(ld, E, &L->proj)) ||
+        (r = joint_bias(ld, J, {{0u, p + "q.b", H * D}, {(uint32_t)(H * D), p + "k.b", G * D}, {(uint32_t)((H + G) * D), p + "v.b", G * VD}}, &L->proj_b))) return r;
+    L->head_norm = true;
+    if ((r = ld.vec(p + "q.norm", {D}, &L->qn)) || (r = ld.vec(p + "k.norm", {D}, &L->kn)) || (r = ld.put_f32(std::vector<float>(H, 0.0f), &L->sink))) return r;
+    return ld.stacked({p + "o"}, {E}, H * VD, &L->o);
+}
+
+// matrix memory: one product gives [q | k | v | output gate | input gate | forget gate], the last two with biases
+int load_memory(Loader &ld, const nb::Json *m, const std::string &p, Layer *L, uint32_t E) {
+    double cap;
+    if (!u32_of(m, "heads", &L->H) || !u32_of(m, "dim", &L->dim) || !u32_of(m, "vdim", &L->vdim) || !m->number("gate_cap", &cap)) return fail(NB200_EINVAL, "%s: an mlstm mixer needs heads, dim, vdim and gate_cap", p.c_str());
+    if (!L->H || !L->dim || !L->vdim || !(cap > 0.0)) return fail(NB200_EINVAL, "%s: heads %u / dim %u / vdim %u / gate_cap %g unusable", p.c_str(), L->H, L->dim, L->vdim, cap);
+    if (L->dim > kMemDim || L->vdim > 4096) return fail(NB200_EINVAL, "%s: dim %u above %u or vdim %u above 4096 has no memory kernel", p.c_str(), L->dim, kMemDim, L->vdim);
+    L->gate_cap = (float)cap;
+    const uint64_t H = L->H, D = L->dim, VD = L->vdim;
+    JointRows J; int r;
+    if ((r = J.add(ld, p + "q", H * D, E, nullptr)) || (r = J.add(ld, p + "k", H * D, E, nullptr)) || (r = J.add(ld, p + "v", H * VD, E, nullptr)) || (r = J.add(ld, p + "g", H * VD, E, nullptr)) ||
+        (r = J.add(ld, p + "i", H, E, &L->c_if)) || (r = J.add(ld, p + "f", H, E, nullptr)) || (r = J.put(ld, E, &L->proj)) ||
+        (r = joint_bias(ld, J, {{L->c_if, p + "i.b", H}, {L->c_if + L->H, p + "f.b", H}}, &L->proj_b)) || (r = ld.vec(p + "norm", {H * VD}, &L->gn))) return r;
+    return ld.stacked({p + "o"}, {E}, H * VD, &L->o);
+}
+
 // grouped-query attention ("left") and gated delta rule ("right") on the same input.  Of the attention, by presence: rot, softcap, the
 // tensors q.norm / k.norm (gains of a norm over the whole projection), sink and g (one gate per head)
 int load_attn_delta(Loader &ld, const nb::Json *m, const std::string &p, Layer *L, uint32_t E, uint32_t positions) {
     const nb::Json *lf = m->get("left"), *rt = m->get("right");
     if (!lf || lf->t != nb::Json::Obj || !rt || rt->t != nb::Json::Obj) return fail(NB200_EINVAL, "%s: a parallel mixer needs left and right", p.c_str());
-    double sc;
-    if (!u32_of(lf, "heads", &L->H) || !u32_of(lf, "kv_heads", &L->G) || !u32_of(lf, "dim", &L->dim) || !u32_of(lf, "vdim", &L->vdim) || !lf->number("scale", &sc))
-        return fail(NB200_EINVAL, "%sleft: an attention needs heads, kv_heads, dim, vdim and scale", p.c_str());
-    L->scale = (float)sc;
-    if (!L->H || !L->G || L->H % L->G || !L->dim || !L->vdim) return fail(NB200_EINVAL, "%sleft: heads %u / kv_heads %u / dim %u / vdim %u unusable", p.c_str(), L->H, L->G, L->dim, L->vdim);
-    if (L->dim > 256 || L->vdim > 256) return fail(NB200_EINVAL, "%sleft: dim %u or vdim %u above 256 has no attention kernel", p.c_str(), L->dim, L->vdim);
     int r;
-    if (lf->present("softcap")) { double c; if (!lf->number("softcap", &c) || !(c >= 0.0)) return fail(NB200_EINVAL, "%sleft: softcap must be a number >= 0", p.c_str()); L->softcap = (float)c; }
-    if (lf->present("rot")) {
-        const nb::Json *rot = lf->get("rot");
-        if (!u32_of(rot, "dims", &L->rot_dims) || L->rot_dims > L->dim || (L->rot_dims & 1u)) return fail(NB200_EINVAL, "%sleft: rot needs an even dims <= dim", p.c_str());
-        if (L->rot_dims && (r = rope_table(ld, rot, p, L->rot_dims, positions, &L->rot_tab))) return r;
-        L->a_half = L->rot_dims / 2u;
-    }
+    if ((r = load_gqa_sizes(ld, lf, p + "left", L, positions))) return r;
     const uint64_t H = L->H, G = L->G, D = L->dim, VD = L->vdim;
-    L->RL = (uint32_t)((G * D + G * VD + 3u) & ~(uint64_t)3u);
     const std::string q = p + "left.";
     JointRows J;
     if ((r = J.add(ld, q + "q", H * D, E, nullptr)) || (r = J.add(ld, q + "k", G * D, E, nullptr)) || (r = J.add(ld, q + "v", G * VD, E, nullptr)) ||
@@ -1271,10 +1355,11 @@ uint32_t gqa_hb(const Layer &L) { return std::min(L.H / L.G, kGqaHeads); }
 int gqa_branch(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx, float *dst) {
     const uint32_t T = cx.T, H = L.H, G = L.G, D = L.dim, VD = L.vdim, P = L.proj.rows;
     GqaArgs a{e->b_p, P, 0u, H * D, H * D + G * D, L.c_hg, L.qn, L.kn, L.rot_tab, L.a_half, run.cache, cx.table, T, H, G, D, VD, L.RL, cx.pos0, cx.pos_ptr, e->eps,
-              L.scale, L.softcap, L.sink, L.has_gate ? 1u : 0u, e->b_a, 1u, e->b_gpart, e->b_gtick, gqa_hb(L)};
+              L.scale, L.softcap, L.sink, L.has_gate ? 1u : 0u, e->b_a, 1u, e->b_gpart, e->b_gtick, gqa_hb(L), L.block_size, L.head_norm ? 1u : 0u};
     int r;
     if (T <= kGemvMaxM) {      // a captured step does not know the position: blocks without a share of the keys leave at once
-        const uint32_t pages = ((cx.pos_ptr ? e->max_tokens : cx.pos0 + T) + kPage - 1u) / kPage;
+        uint32_t pages = ((cx.pos_ptr ? e->max_tokens : cx.pos0 + T) + kPage - 1u) / kPage;
+        if (L.block_size) pages = std::min(pages, (L.block_size + kPage - 2u) / kPage + 1u);      // a block of positions may start inside a page
         a.nsplit = std::max(1u, std::min(kGqaSplitMax, pages));
         const dim3 grid(a.nsplit, G * ((H / G + a.hb - 1u) / a.hb), T), block(256);
         const size_t smem = gqa_decode_smem(D, VD);
@@ -1302,8 +1387,51 @@ int mix_attn_delta(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &
     return 0;
 }
 
+int mix_gqa(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) {
+    int r;
+    return (r = gemm(e, plain(e->hm, e->E, L.proj, e->b_p, L.proj.rows, cx.T, L.proj_b), 1, cx.T)) ? r : gqa_branch(e, L, run, cx, e->d);
+}
+
+// ---- matrix memory ----
+// one product gives [q | k | v | g | i | f]; short portions: the rest up to the output product is one kernel; long ones: gates, states
+// before every chunk, outputs of all chunks, norm and gate
+int mix_memory(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) {
+    const uint32_t T = cx.T, H = L.H, D = L.dim, VD = L.vdim, P = L.proj.rows, k0 = H * D, v0 = 2 * H * D, g0 = v0 + H * VD, i0 = L.c_if, f0 = i0 + H;
+    const float qscale = (float)(1.0 / sqrt((double)D));
+    float *S = cx.st + run.st_S, *n = cx.st + run.st_n, *m = cx.st + run.st_m;
+    int r;
+    if ((r = gemm(e, plain(e->hm, e->E, L.proj, e->b_p, P, T, L.proj_b), 1, T))) return r;
+    if (T <= kGemvMaxM) {
+        MemStepArgs a{e->b_p, P, 0u, k0, v0, g0, i0, f0, L.gate_cap, qscale, e->eps, L.gn, S, n, m, e->b_a, T, H, D, VD};
+        const uint32_t nb = memory_step_blocks(VD), want = std::max(128u, memory_step_cols(VD) * 8u);
+#define MEM_STEP(DCH) launch<MemStepArgs>(e, k_memory_step<DCH>, dim3(nb, H), dim3(std::min(kMemThreads, want)), memory_step_smem(DCH, VD), a, nb)
+        if (D <= 32) r = MEM_STEP(1);
+        else if (D <= 64) r = MEM_STEP(2);
+        else if (D <= 128) r = MEM_STEP(4);
+        else if (D <= 256) r = MEM_STEP(8);
+        else r = MEM_STEP(16);
+#undef MEM_STEP
+        return r ? r : gemm(e, plain(e->b_a, H * VD, L.o, e->d, e->E, T), 1, T);
+    }
+    const uint32_t chunks = (T + kMemChunk - 1u) / kMemChunk;
+    MemGatesArgs ga{e->b_p, P, i0, f0, L.gate_cap, m, e->b_mfa, e->b_mfb, e->b_mfc, e->b_mmt, e->b_mme, T, H, chunks};
+    MemStatesArgs sa{e->b_p, P, k0, v0, e->b_mfb, e->b_mfc, e->b_mme, S, n, e->b_mS, e->b_mn, T, H, D, VD, chunks};
+    MemOutArgs oa{e->b_p, P, 0u, k0, v0, qscale, e->b_mfa, e->b_mfb, e->b_mmt, e->b_mme, e->b_mS, e->b_mn, e->b_mo, T, H, D, VD, chunks};
+    if ((r = launch<MemGatesArgs>(e, k_memory_gates, dim3(H), dim3(1024), 0, ga)) ||
+        (r = launch<MemStatesArgs>(e, k_memory_states, dim3((VD + 31u) / 32u, (D + 63u) / 64u, H), dim3(256), 0, sa))) return r;
+    // 128 value columns per block (the scores are made once for them) where that still fills the GPU twice
+    if (VD > 64u && (VD + 127u) / 128u * chunks * H >= 2u * (uint32_t)e->num_sms) r = launch<MemOutArgs>(e, k_memory_out<2>, dim3((VD + 127u) / 128u, chunks, H), dim3(256), memory_out_smem(2), oa);
+    else r = launch<MemOutArgs>(e, k_memory_out<1>, dim3((VD + 63u) / 64u, chunks, H), dim3(256), memory_out_smem(1), oa);
+    if (r) return r;
+    RetOutArgs na{e->b_mo, e->b_p + g0, P, e->b_a, T, H, VD, e->eps, L.gn, 1u, VD};
+    if ((r = launch<RetOutArgs>(e, k_retention_out, dim3((T * H + 7u) / 8u), dim3(256), 0, na))) return r;
+    return gemm(e, plain(e->b_a, H * VD, L.o, e->d, e->E, T), 1, T);
+}
+
 int mix(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) {
     switch (L.type) {
+        case MIX_GQA: return mix_gqa(e, L, run, cx);
+        case MIX_MEMORY: return mix_memory(e, L, run, cx);
         case MIX_DELTA: return mix_delta(e, L, run, cx);
         case MIX_ATTN_DELTA: return mix_attn_delta(e, L, run, cx);
         case MIX_RGLRU: return mix_rglru(e, L, run, cx);
@@ -1393,10 +1521,10 @@ int dyt_residual(LayeredEngine *e, const Layer *moe, const Dyt &post, const Dyt 
     return launch<DytResArgs>(e, k_dyt_residual, dim3(ew_grid((size_t)T * e->E)), dim3(256), 0, a);
 }
 
-// dense feed-forward with the exact gelu as the first product's epilogue: e->h2 -> e->d
-int ff_dense_gelu(LayeredEngine *e, const Layer &L, uint32_t T) {
+// dense feed-forward with the activation (exact gelu, squared relu) as the first product's epilogue: e->h2 -> e->d
+int ff_dense_act(LayeredEngine *e, const Layer &L, uint32_t T) {
     int r;
-    if ((r = gemm(e, plain(e->h2, e->E, L.up, e->b_f, L.ff, T, nullptr, EPI_GELU_ERF), 1, T))) return r;
+    if ((r = gemm(e, plain(e->h2, e->E, L.up, e->b_f, L.ff, T, nullptr, L.ff_kind == FF_DENSE_RELU2 ? EPI_RELU2 : EPI_GELU_ERF), 1, T))) return r;
     return gemm(e, plain(e->b_f, L.ff, L.down, e->d, e->E, T), 1, T);
 }
 
@@ -1441,6 +1569,35 @@ int post_norm(LayeredEngine *e, const Layer *two, const float *w, float *keep, u
     return launch<PostNormArgs>(e, k_post_norm<0>, dim3(T), dim3(threads), 0, a);
 }
 
+// the routed squared-relu experts: e->h2 -> the rows of e->b_eo (one per token and choice, in expert order), their weights in e->b_wt
+int ff_moe_relu2(LayeredEngine *e, const Layer &L, uint32_t T) {
+    const uint32_t E = e->E;
+    int r;
+    RouteArgs ra{e->h2, L.router, e->b_idx, e->b_wt, e->b_cnt, e->b_off, e->b_fill, e->b_slot, e->b_rows, T, L.NE, L.top, E, L.route_mode};
+    ra.groups = L.groups; ra.keep = L.keep_groups; ra.wscale = L.route_scale;
+    if (T <= kGemvMaxM) { if ((r = launch<RouteArgs>(e, k_route_small, dim3(1), dim3(1024), route_smem(L.NE, 1024), ra))) return r; }
+    else if ((r = launch<RouteArgs>(e, k_route, dim3(T), dim3(256), route_smem(L.NE, 256), ra)) ||
+             (r = launch<RouteArgs>(e, k_route_place, dim3(1), dim3(1024), 0, ra))) return r;
+    GemmArgs u{};
+    u.A = e->h2; u.lda = E; u.W = L.up.p; u.ldw = E; u.C = e->b_hb; u.ldc = L.ff; u.M = T; u.N = L.ff; u.K = E; u.a_gmod = 1;
+    u.g_off = e->b_off; u.a_rows = e->b_rows; u.w_gstride = (uint64_t)L.ff * E; u.epi = EPI_RELU2;
+    if ((r = gemm(e, u, L.NE, T, false, T * L.top))) return r;
+    GemmArgs dn{};
+    dn.A = e->b_hb; dn.lda = L.ff; dn.W = L.down.p; dn.ldw = L.ff; dn.C = e->b_eo; dn.ldc = E; dn.M = T; dn.N = E; dn.K = L.ff; dn.a_gmod = 1;
+    dn.g_off = e->b_off; dn.w_gstride = (uint64_t)E * L.ff;
+    return gemm(e, dn, L.NE, T, false, T * L.top);
+}
+
+// x = rms_norm(alpha x + sublayer output) w; moe: the output is the chosen experts' rows, else e->d
+int post_ln(LayeredEngine *e, const Layer *moe, const float *w, float *keep, uint32_t T) {
+    PostLnArgs a{e->x, e->d, moe ? e->b_eo : nullptr, e->b_slot, e->b_wt, moe ? moe->top : 0u, w, e->alpha, keep, T, e->E, e->eps};
+    // a short portion is a few lone blocks: wide ones, so that a thread's chain of loads stays short
+    const uint32_t per = T <= kGemvMaxM ? 2u : 8u, threads = std::min(1024u, std::max(128u, (e->E / per + 31u) & ~31u));
+    if (e->E <= 2u * threads) return launch<PostLnArgs>(e, k_post_ln<2>, dim3(T), dim3(threads), 0, a);
+    if (e->E <= 8u * threads) return launch<PostLnArgs>(e, k_post_ln<8>, dim3(T), dim3(threads), 0, a);
+    return launch<PostLnArgs>(e, k_post_ln<0>, dim3(T), dim3(threads), 0, a);
+}
+
 // every layer run over T tokens (x already holds their embeddings) of the sequence in `slot`, whose first token sits at pos0
 // (+ *pos_ptr: a captured decode step keeps the position on the device and uses a fixed number of key splits)
 int run_layers(LayeredEngine *e, uint32_t slot, uint32_t T, uint32_t pos0, const uint32_t *pos_ptr = nullptr) {
@@ -1458,6 +1615,13 @@ int run_layers(LayeredEngine *e, uint32_t slot, uint32_t T, uint32_t pos0, const
             if (L.has_mlp && ((r = ff_glu_dense(e, L, T)) || (r = post_norm(e, nullptr, L.pn2, keep, T)))) return r;
             continue;
         }
+        if (e->form == FORM_POST_LN) {      // sublayers read x itself, and the sum is normed
+            if ((r = mix(e, L, run, cx)) || (r = post_ln(e, nullptr, L.pn1, L.has_mlp ? nullptr : keep, T))) return r;
+            if (!L.has_mlp) continue;
+            const bool moe = L.ff_kind == FF_MOE;
+            if ((r = moe ? ff_moe_relu2(e, L, T) : ff_dense_act(e, L, T)) || (r = post_ln(e, moe ? &L : nullptr, L.pn2, keep, T))) return r;
+            continue;
+        }
         if (e->form == FORM_HYPER) {
             // e->hm already holds the mixer's input (from the embedding step or the update before); every update also prepares the
             // input of the sublayer that follows (this layer's feed-forward, or the next run's mixer)
@@ -1466,7 +1630,7 @@ int run_layers(LayeredEngine *e, uint32_t slot, uint32_t T, uint32_t pos0, const
             if (!L.has_mlp) { if ((r = hc_step(e, L.hc1, L.ls1, nullptr, NX ? NX->hc1 : nullptr, NX ? NX->ln1 : nullptr, e->hm, keep, T))) return r; continue; }
             if ((r = hc_step(e, L.hc1, L.ls1, nullptr, L.hc2, L.ln2, e->h2, nullptr, T))) return r;
             const bool moe = L.ff_kind == FF_MOE_SCORED;
-            if ((r = moe ? ff_moe_scored(e, L, T) : ff_dense_gelu(e, L, T))) return r;
+            if ((r = moe ? ff_moe_scored(e, L, T) : ff_dense_act(e, L, T))) return r;
             if ((r = hc_step(e, L.hc2, L.ls2, moe ? &L : nullptr, NX ? NX->hc1 : nullptr, NX ? NX->ln1 : nullptr, e->hm, keep, T))) return r;
             continue;
         }
@@ -1518,18 +1682,7 @@ int run_layers(LayeredEngine *e, uint32_t slot, uint32_t T, uint32_t pos0, const
             // The layer is parallel: the feed-forward reads h2 = norm2(x) of the SAME x and shares no buffer with the mixer, so its
             // kernels go to a second stream (a parallel branch of the captured decode graph) and join before the residual update.
             if (e->branch_streams) { e->cur = e->side; CK(cudaStreamWaitEvent(e->side, e->ev_fork, 0)); }
-            RouteArgs ra{e->h2, L.router, e->b_idx, e->b_wt, e->b_cnt, e->b_off, e->b_fill, e->b_slot, e->b_rows, T, L.NE, L.top, E};
-            if (T <= kGemvMaxM) { if ((r = launch<RouteArgs>(e, k_route_small, dim3(1), dim3(1024), route_smem(L.NE, 1024), ra))) return r; }
-            else if ((r = launch<RouteArgs>(e, k_route, dim3(T), dim3(256), route_smem(L.NE, 256), ra)) ||
-                     (r = launch<RouteArgs>(e, k_route_place, dim3(1), dim3(1024), 0, ra))) return r;
-            GemmArgs u{};
-            u.A = e->h2; u.lda = E; u.W = L.up.p; u.ldw = E; u.C = e->b_hb; u.ldc = L.ff; u.M = T; u.N = L.ff; u.K = E; u.a_gmod = 1;
-            u.g_off = e->b_off; u.a_rows = e->b_rows; u.w_gstride = (uint64_t)L.ff * E; u.epi = EPI_RELU2;
-            if ((r = gemm(e, u, L.NE, T, false, T * L.top))) return r;
-            GemmArgs dn{};
-            dn.A = e->b_hb; dn.lda = L.ff; dn.W = L.down.p; dn.ldw = L.ff; dn.C = e->b_eo; dn.ldc = E; dn.M = T; dn.N = E; dn.K = L.ff; dn.a_gmod = 1;
-            dn.g_off = e->b_off; dn.w_gstride = (uint64_t)E * L.ff;
-            if ((r = gemm(e, dn, L.NE, T, false, T * L.top))) return r;
+            if ((r = ff_moe_relu2(e, L, T))) return r;
             if (L.has_shared) {      // a third branch: the shared expert depends on h2 only
                 if (e->branch_streams) { e->cur = e->side2; CK(cudaStreamWaitEvent(e->side2, e->ev_fork, 0)); }
                 if ((r = gemm(e, plain(e->h2, E, L.sup, e->b_sh, L.sff, T, nullptr, EPI_RELU2), 1, T)) || (r = gemm(e, plain(e->b_sh, L.sff, L.sdown, e->b_so, E, T), 1, T))) return r;
@@ -1565,8 +1718,8 @@ int embed_tokens(LayeredEngine *e, uint32_t slot, const uint32_t *tok_dev, uint3
         e->launches++;
         return 0;
     }
-    if (e->f32) k_embed<float><<<T, 128, 0, e->stream>>>(tok_dev, pos_ptr, (const float *)e->embed.p, e->x, e->keep_x0 ? e->x0 : nullptr, e->E);
-    else k_embed<__nv_bfloat16><<<T, 128, 0, e->stream>>>(tok_dev, pos_ptr, (const __nv_bfloat16 *)e->embed.p, e->x, e->keep_x0 ? e->x0 : nullptr, e->E);
+    if (e->f32) k_embed<float><<<T, 128, 0, e->stream>>>(tok_dev, pos_ptr, (const float *)e->embed.p, e->x, e->keep_x0 ? e->x0 : nullptr, e->E, e->emb_scale);
+    else k_embed<__nv_bfloat16><<<T, 128, 0, e->stream>>>(tok_dev, pos_ptr, (const __nv_bfloat16 *)e->embed.p, e->x, e->keep_x0 ? e->x0 : nullptr, e->E, e->emb_scale);
     CK(cudaGetLastError());
     e->launches++;
     return 0;
@@ -1586,10 +1739,12 @@ int head_rows(LayeredEngine *e, uint32_t nw, const uint32_t *want_dev = nullptr)
         e->launches++;
         return gemm(e, plain(e->b_xn, e->E, e->head, e->logits, e->V, nw), 1, nw);
     }
-    k_final_norm<<<nw, 256, 0, e->stream>>>(e->x, want_dev ? want_dev : e->want_dev, e->final_norm, e->b_xn, e->E, e->eps, e->form == FORM_SANDWICH ? 1u : e->form == FORM_POST ? 2u : 0u);
+    k_final_norm<<<nw, 256, 0, e->stream>>>(e->x, want_dev ? want_dev : e->want_dev, e->final_norm, e->b_xn, e->E, e->eps, e->form == FORM_SANDWICH ? 1u : e->form == FORM_POST || e->form == FORM_POST_LN ? 2u : 0u);
     CK(cudaGetLastError());
     e->launches++;
-    return gemm(e, plain(e->b_xn, e->E, e->head, e->logits, e->V, nw), 1, nw);
+    GemmArgs hd = plain(e->b_xn, e->E, e->head, e->logits, e->V, nw, nullptr, e->logit_cap > 0.0f ? EPI_SOFTCAP : EPI_NONE);
+    hd.cap = e->logit_cap;
+    return gemm(e, hd, 1, nw);
 }
 
 // One decode step of `slot`: the token ids_dev[*dpos] at position *dpos, logits of it in e->logits[0..V).  The position lives in
@@ -1976,7 +2131,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
     int r;
     const nb::Json *arch = cfg.get("architecture");
     const std::string design = arch && arch->t == nb::Json::Str ? arch->str : "";
-    e->form = design == "Rakarax" || design == "Gokinex" ? FORM_SANDWICH : design == "Vumunex" ? FORM_HYPER : design == "Kadesun" ? FORM_POST : FORM_PARALLEL_SHIFT;
+    e->form = design == "Rakarax" || design == "Gokinex" ? FORM_SANDWICH : design == "Vumunex" ? FORM_HYPER : design == "Kadesun" ? FORM_POST : design == "Fidatar" ? FORM_POST_LN : FORM_PARALLEL_SHIFT;
     e->norm_kind = design == "Gokinex" ? NORM_DYT : NORM_RMS_ZERO;
     if ((r = ld.stacked({"embed"}, {e->V}, E, &e->embed)) || (r = ld.stacked({"head"}, {e->V}, E, &e->head))) return r;
     e->layers.resize(NL);
@@ -2042,7 +2197,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
                 const nb::Json *f = lj.get("mlp"), *kind = f->get("kind");
                 if ((r = ld.vec(p + "norm2", {E}, &L.ln2)) || (r = load_hc(ld, p + "hc2.", e->S, &L.hc2))) return r;
                 if (dir->tensors.count(p + "ls2") && (r = ld.vec(p + "ls2", {E}, &L.ls2))) return r;
-                if (kind && kind->t == nb::Json::Str && kind->str == "dense") r = load_dense_gelu(ld, f, p + "mlp.", &L, E);
+                if (kind && kind->t == nb::Json::Str && kind->str == "dense") r = load_dense_act(ld, f, p + "mlp.", &L, E, FF_DENSE_GELU);
                 else if (kind && kind->t == nb::Json::Str && kind->str == "moe") r = load_moe_scored(ld, f, p + "mlp.", &L, E, true);
                 else return fail(NB200_EINVAL, "layer %u: feed-forward kind \"%s\" is not known", i, kind && kind->t == nb::Json::Str ? kind->str.c_str() : "?");
                 if (r) return r;
@@ -2067,6 +2222,35 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
                 const nb::Json *f = lj.get("mlp"), *kind = f->get("kind");
                 if (!kind || kind->t != nb::Json::Str || kind->str != "dense") return fail(NB200_EINVAL, "layer %u: feed-forward kind \"%s\" is not known here", i, kind && kind->t == nb::Json::Str ? kind->str.c_str() : "?");
                 if ((r = ld.vec(p + "norm2", {E}, &L.pn2)) || (r = load_glu_dense(ld, f, p + "mlp.", &L, E, 2u))) return r;
+            }
+        }
+    } else if (e->form == FORM_POST_LN) {
+        const nb::Json *emb = cfg.get("embedding");
+        double sc = 1.0, alpha = 1.0, cap = 0.0;
+        if (emb && emb->t == nb::Json::Obj && emb->present("scale") && !emb->number("scale", &sc)) return fail(NB200_EINVAL, "embedding.scale must be a number");
+        if (cfg.present("postln_alpha") && !cfg.number("postln_alpha", &alpha)) return fail(NB200_EINVAL, "postln_alpha must be a number");
+        if (cfg.present("logit_softcap") && (!cfg.number("logit_softcap", &cap) || !(cap >= 0.0))) return fail(NB200_EINVAL, "logit_softcap must be a number >= 0");
+        e->emb_scale = (float)sc; e->alpha = (float)alpha; e->logit_cap = (float)cap;
+        if ((r = ld.vec("final.norm", {E}, &e->final_norm))) return r;
+        const uint32_t page_tokens = ((max_tokens + kPage - 1) / kPage + std::max(1u, env_u32("NB200_MAX_SEQS", 8))) * kPage;      // every position the cache pages can hold
+        for (uint32_t i = 0; i < NL; i++) {
+            Run q; q.layer = i; e->runs.push_back(q);
+            const nb::Json &lj = layers->arr[i];
+            Layer &L = e->layers[i];
+            const std::string p = "l" + std::to_string(i) + ".";
+            const nb::Json *type = lj.get("type"), *mixer = lj.get("mixer");
+            if (!type || type->t != nb::Json::Str || !mixer || mixer->t != nb::Json::Obj) return fail(NB200_EINVAL, "layer %u needs \"type\" and \"mixer\"", i);
+            if ((r = ld.vec(p + "norm1", {E}, &L.pn1))) return r;
+            if (type->str == "attention") { L.type = MIX_GQA; r = load_gqa(ld, mixer, p + "mix.", &L, E, page_tokens); }
+            else if (type->str == "mlstm") { L.type = MIX_MEMORY; r = load_memory(ld, mixer, p + "mix.", &L, E); }
+            else return fail(NB200_EINVAL, "layer %u: mixer type \"%s\" is not known", i, type->str.c_str());
+            if (r) return r;
+            if (lj.present("mlp")) {
+                const nb::Json *f = lj.get("mlp"), *kind = f->get("kind");
+                if ((r = ld.vec(p + "norm2", {E}, &L.pn2))) return r;
+                if (kind && kind->t == nb::Json::Str && kind->str == "dense") r = load_dense_act(ld, f, p + "mlp.", &L, E, FF_DENSE_RELU2);
+                else r = load_moe(ld, f, p + "mlp.", &L, E, true);
+                if (r) return r;
             }
         }
     } else if (e->form == FORM_SANDWICH) {
@@ -2164,6 +2348,16 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
                 q.st_S = off; off += (size_t)L.dH * L.dVD * L.dD;
                 if (L.type == MIX_ATTN_DELTA) { DM(q.cache, (size_t)e->n_pages * kPage * L.RL * 4); CK(cudaMemset(q.cache, 0, (size_t)e->n_pages * kPage * L.RL * 4)); }
                 break;
+            case MIX_GQA:            // rows of [normed and turned keys | values]
+                DM(q.cache, (size_t)e->n_pages * kPage * L.RL * 4);
+                CK(cudaMemset(q.cache, 0, (size_t)e->n_pages * kPage * L.RL * 4));
+                break;
+            case MIX_MEMORY:         // the state [head][value column][key coordinate], the normaliser [head][key coordinate], the running maximum
+                off = (off + 3) & ~(size_t)3;
+                q.st_S = off; off += (size_t)L.H * L.vdim * L.dim;
+                q.st_n = off; off += (size_t)L.H * L.dim;
+                q.st_m = off; off += L.H;
+                break;
             case MIX_RETENTION: q.st_S = off; off += (size_t)L.H * L.vdim * L.dim; break;
             default:          // window attention + selective scan: the tails of both convolutions, the scan state, a cache of key/value rows
                 q.st_conv = off; off += (size_t)(L.a_taps - 1) * (L.H + L.G) * L.dim;
@@ -2187,6 +2381,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
     uint32_t sP = 0, sQK = 0, sXC = 0, sA = 0, sRO = 0, sDBC = 0, sF = 0;
     uint32_t sDP = 0, sDT = 0, sXC2 = 0, sY = 0, sF2 = 0; size_t sSS = 0, diff_smem[4] = {0, 0, 0, 0};      // differential attention, state-space duality, gated feed-forward
     uint32_t dC = 0, dV = 0, dBlk = 0, dSp = 0, dGt = 0, dPart = 0, dTick = 0; size_t gqa_smem[5] = {0, 0, 0, 0, 0};      // gated delta rule, grouped-query attention
+    uint32_t mMH = 0, mMO = 0, mMD = 0; size_t mMS = 0;      // matrix memory
     size_t win_smem[4] = {0, 0, 0, 0};      // most shared memory any layer asks of the window-attention instances, per value-column count
     for (const Run &q : e->runs) {
         const Layer &L = e->layers[q.layer];
@@ -2199,7 +2394,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
             size_t &sm = win_smem[L.dim <= 32 ? 0 : L.dim <= 64 ? 1 : L.dim <= 128 ? 2 : 3];
             sm = std::max(sm, std::max(win_attn_smem(L.H, L.dim, L.RL, qt), win_attn_smem(L.H, L.dim, L.RL, 1)));
         }
-        if (L.ff_kind == FF_DENSE_POLY || L.ff_kind == FF_DENSE_GELU) sF = std::max(sF, L.ff);
+        if (L.ff_kind == FF_DENSE_POLY || L.ff_kind == FF_DENSE_GELU || L.ff_kind == FF_DENSE_RELU2) sF = std::max(sF, L.ff);
         if (L.type == MIX_DIFF_ATTN) {
             sP = std::max(sP, L.H * 2 * L.dim + (L.kv_from < 0 ? L.G * (2 * L.dim + L.vdim) : 0u)); sA = std::max(sA, L.H * L.vdim);
             sDP = std::max(sDP, L.H * 2 * (L.vdim + 2)); sDT = std::max(sDT, (L.H + L.a_hpb1 - 1) / L.a_hpb1);
@@ -2218,7 +2413,12 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
             if (L.ra) dSp = std::max(dSp, L.dH * L.dD);
             if (L.rg) dGt = std::max(dGt, L.dH * L.dVD);
         }
-        if (L.type == MIX_ATTN_DELTA) {
+        if (L.type == MIX_MEMORY) {
+            sP = std::max(sP, L.proj.rows); sA = std::max(sA, L.H * L.vdim); mMH = std::max(mMH, L.H); mMO = std::max(mMO, L.H * L.vdim); mMD = std::max(mMD, L.H * L.dim);
+            mMS = std::max(mMS, (size_t)L.H * L.vdim * L.dim);
+        }
+        if (L.type == MIX_GQA) sP = std::max(sP, L.proj.rows);
+        if (L.type == MIX_ATTN_DELTA || L.type == MIX_GQA) {
             sA = std::max(sA, L.H * L.vdim); dPart = std::max(dPart, L.H * (L.vdim + 2)); dTick = std::max(dTick, L.G * ((L.H / L.G + gqa_hb(L) - 1u) / gqa_hb(L)));
             const int vj = gqa_vj(L.vdim);
             if (gqa_attn_smem(L.dim, vj) > kGqaSmemMax) return fail(NB200_EINVAL, "attention with %u query/key and %u value coordinates does not fit the attention kernel's shared memory", L.dim, L.vdim);
@@ -2241,8 +2441,14 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
         if (dSp) DM(e->b_gsp, T * dSp * 4);
         if (dGt) DM(e->b_gt, T * dGt * 4);
     }
+    if (mMH) {
+        const size_t chunks = (T + kMemChunk - 1) / kMemChunk;
+        DM(e->b_mfa, mMH * T * 8); DM(e->b_mfb, mMH * T * 8); DM(e->b_mfc, mMH * chunks * 8); DM(e->b_mmt, mMH * T * 4); DM(e->b_mme, mMH * (chunks + 1) * 4);
+        DM(e->b_mS, chunks * mMS * 4); DM(e->b_mn, chunks * mMD * 4); DM(e->b_mo, T * mMO * 4);
+        CK(cudaFuncSetAttribute((const void *)k_memory_out<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)memory_out_smem(2)));
+    }
     if (dPart) {
-        DM(e->d2, T * E * 4); DM(e->b_gpart, (size_t)kGemvMaxM * kGqaSplitMax * dPart * 4); DM(e->b_gtick, (size_t)kGemvMaxM * dTick * 4);
+        if (dC) DM(e->d2, T * E * 4); DM(e->b_gpart, (size_t)kGemvMaxM * kGqaSplitMax * dPart * 4); DM(e->b_gtick, (size_t)kGemvMaxM * dTick * 4);
         CK(cudaMemset(e->b_gtick, 0, (size_t)kGemvMaxM * dTick * 4));
         if (gqa_smem[1] > 48 * 1024) CK(cudaFuncSetAttribute((const void *)k_gqa_attn<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gqa_smem[1]));
         if (gqa_smem[2] > 48 * 1024) CK(cudaFuncSetAttribute((const void *)k_gqa_attn<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gqa_smem[2]));
@@ -2289,7 +2495,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
     }
     if (e->form == FORM_HYPER) DM(e->xs, (size_t)e->S * T * E * 4);
     DM(e->x, T * E * 4); DM(e->d, T * E * 4);
-    if (e->form == FORM_POST) { e->hm = e->x; e->h2 = e->x; }      // no input norms: a sublayer reads the residual
+    if (e->form == FORM_POST || e->form == FORM_POST_LN) { e->hm = e->x; e->h2 = e->x; }      // no input norms: a sublayer reads the residual
     else { DM(e->hm, T * E * 4); DM(e->h2, T * E * 4); }
     if (e->keep_x0) DM(e->x0, T * E * 4);
     if (mC) { DM(e->b_yx, T * 2 * mC * 4); DM(e->b_u, T * mC * 4); DM(e->b_g, T * 2 * mC * 4); DM(e->b_sy, T * mC * 4); }

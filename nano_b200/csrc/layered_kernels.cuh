@@ -22,7 +22,7 @@
 //                        k_combine (weighted sum in choice order + shared expert + mixer output -> residual)
 //
 // More mechanisms (position table, sandwich norms, rotary positions, retention, window attention, selective scan, PolyNorm) live in
-// layered_mixers.cuh and layered_mixers2 / 3 / 4.cuh under the same rules.
+// layered_mixers.cuh and layered_mixers2 / 3 / 4 / 5.cuh under the same rules.
 //
 // What is fp32 here regardless of the weight type: the residual stream, every norm, router logits, attention scores / weights /
 // accumulators, gates, decays and the recurrent state.  bf16 enters only as a matrix-product operand.
@@ -40,7 +40,7 @@ constexpr uint32_t kAttnWarps = 8;        // heads per attention block
 constexpr uint32_t kGemvMaxM = 4;         // rows a k_gemv launch handles per group
 
 enum CMode : uint32_t { C_ADD = 1, C_SCALE = 2 };
-enum Epi : uint32_t { EPI_NONE = 0, EPI_BIAS = 1, EPI_GELU_SPLIT = 2, EPI_SIGMOID = 3, EPI_RELU2 = 4, EPI_GELU_CONV = 5, EPI_SOFTPLUS = 6, EPI_CONV_RANGES = 7, EPI_SIGMOID_TAIL = 8, EPI_GELU_ERF = 9 };
+enum Epi : uint32_t { EPI_NONE = 0, EPI_BIAS = 1, EPI_GELU_SPLIT = 2, EPI_SIGMOID = 3, EPI_RELU2 = 4, EPI_GELU_CONV = 5, EPI_SOFTPLUS = 6, EPI_CONV_RANGES = 7, EPI_SIGMOID_TAIL = 8, EPI_GELU_ERF = 9, EPI_SOFTCAP = 10 };
 
 // C[r, c0 + n] = epi( sum_k A[arow(r), a0 + k] * W[g][n, k] + bias[g][n] )   for the rows r of group g
 //   rows of group g : [g_off[g], g_off[g+1])  when g_off is given (sizes known on the device only), else [0, M)
@@ -86,6 +86,8 @@ struct GemmArgs {
     const float *mul; uint32_t ldm;
     // Gated pair, glu 3: the clamped unit  g' = min(g, glu_limit), u' = clamp(u, -glu_limit, glu_limit),  g' sigmoid(1.702 g') (u' + 1).
     float glu_limit;
+    // EPI_SOFTCAP: cap tanh(v / cap)
+    float cap;
 };
 
 // Programmatic dependent launch: every kernel first lets the NEXT kernel of its stream be scheduled (its blocks then sit in their own
@@ -125,6 +127,7 @@ __device__ __forceinline__ float epilogue(float v, const GemmArgs &a, const floa
         case EPI_RELU2: { const float r = fmaxf(v, 0.0f); return r * r; }
         case EPI_SOFTPLUS: return softplusf_(v);
         case EPI_SIGMOID_TAIL: return n >= a.split ? sigmoidf_(v) : v;
+        case EPI_SOFTCAP: return a.cap * tanhf(v / a.cap);
         case EPI_GELU_ERF: return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
         default: return v;
     }
@@ -572,16 +575,16 @@ __device__ __forceinline__ float block_sum(float v, float *red) {
     return s;
 }
 
-// x[t] = embed[tokens[base + t]]; x0 keeps a copy when a later pass adds the embedding output again.  base = *pos_ptr when given: a
+// x[t] = scale embed[tokens[base + t]]; x0 keeps a copy when a later pass adds the embedding output again.  base = *pos_ptr when given: a
 // captured decode step reads "the token at the sequence's present position" without a host-side argument
 template <typename WT>
 __global__ void k_embed(const uint32_t *__restrict__ tokens, const uint32_t *__restrict__ pos_ptr, const WT *__restrict__ embed, float *__restrict__ x,
-                        float *__restrict__ x0, uint32_t E) {
+                        float *__restrict__ x0, uint32_t E, float scale) {
     pdl_enter();
     const uint32_t t = blockIdx.x;
     const WT *src = embed + (size_t)tokens[t + (pos_ptr ? *pos_ptr : 0u)] * E;
     for (uint32_t i = threadIdx.x; i < E; i += blockDim.x) {
-        const float v = wval(src + i);
+        const float v = wval(src + i) * scale;
         x[(size_t)t * E + i] = v;
         if (x0) x0[(size_t)t * E + i] = v;
     }
@@ -1039,12 +1042,14 @@ __global__ void __launch_bounds__(kAttnWarps * 32, attn_two_blocks(RCH, QT, EXAC
 // `top` largest (ties: the lower expert index first) and their weights = softmax over the chosen logits only; counts[e] += 1 per
 // choice.  Dynamic shared memory: route_smem(NE, threads) bytes.
 // mode 0: weights = softmax over the chosen logits; mode 1: weights = sigmoid of the chosen logits, taken as they are (they need not sum to 1);
-// mode 2: scores = softmax over ALL experts, weights = the chosen experts' scores divided by their sum (+ 1e-20).
+// mode 2: scores = softmax over ALL experts, weights = the chosen experts' scores divided by their sum (+ 1e-20);
+// mode 3: scores = sigmoid of the logits; the experts form `groups` equal runs of neighbours, a group's score is the sum of its two
+// largest, and only experts of the `keep` best groups (ties: the lower group) can be chosen; weights = the chosen scores times wscale.
 // extra: the router matrix carries that many more rows after the experts'; their logits go to extra_out [T][extra] and take no part
 // in the choice (a gate of a shared expert, computed with the router's precision).  wrow (optional): the weights once more in
 // expert-sorted row order, wrow[slot[t][j]] = wt[t][j], for a product that scales its rows.
 struct RouteArgs { const float *h; const float *router; uint32_t *idx; float *wt; uint32_t *counts; uint32_t *off; uint32_t *fill; uint32_t *slot; uint32_t *rows; uint32_t T, NE, top, E;
-                   uint32_t mode, extra; float *extra_out; float *wrow; };
+                   uint32_t mode, extra; float *extra_out; float *wrow; uint32_t groups, keep; float wscale; };
 // dynamic shared memory of k_route / k_route_small launched with `threads` threads (NE: rows of the router matrix, extra ones included)
 inline size_t route_smem(uint32_t NE, uint32_t threads) { const uint32_t nw = threads / 32u; return ((size_t)NE + (size_t)NE * (nw > NE ? nw / NE : 1u)) * 4; }
 // router logits of token t into z[NE].  The blockDim/32 warps are dealt out as `ns` slices per expert (ns = warps / NE, at least 1):
@@ -1077,28 +1082,63 @@ __device__ __forceinline__ void route_logits(const RouteArgs &a, uint32_t t, flo
     for (uint32_t e = threadIdx.x; e < NL; e += blockDim.x) {
         float v = 0.0f;
         for (uint32_t sl = 0; sl < ns; sl++) v += zp[e * ns + sl];
-        z[e] = v;
+        z[e] = a.mode == 3u && e < a.NE ? sigmoidf_(v) : v;
     }
 }
-// one thread: the `top` largest of z (ties: the lower index first; z is consumed) and the softmax over them
-__device__ __forceinline__ void route_pick(const RouteArgs &a, uint32_t t, float *z) {
+// one warp: the index of the largest of z[0..n) (ties: the lower index); every lane gets it and the value
+__device__ __forceinline__ uint32_t warp_argmax(const float *z, uint32_t n, uint32_t lane, float *value) {
+    float best = -INFINITY; uint32_t bi = 0xffffffffu;
+    for (uint32_t e = lane; e < n; e += 32u) { const float v = z[e]; if (bi == 0xffffffffu || v > best) { best = v; bi = e; } }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, best, o); const uint32_t oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (oi != 0xffffffffu && (bi == 0xffffffffu || ov > best || (ov == best && oi < bi))) { best = ov; bi = oi; }
+    }
+    *value = best;
+    return bi;
+}
+// one warp: the `top` largest of z (ties: the lower index first; z is consumed) and their weights.  zg: NE floats of scratch
+__device__ __forceinline__ void route_pick(const RouteArgs &a, uint32_t t, float *z, float *zg) {
     uint32_t *idx = a.idx + (size_t)t * a.top; float *wt = a.wt + (size_t)t * a.top;
+    const uint32_t lane = threadIdx.x & 31u;
     float zmax = -INFINITY, zden = 0.0f;
     if (a.mode == 2u) {      // softmax over ALL experts: its maximum and denominator, before the choice consumes z
-        for (uint32_t e = 0; e < a.NE; e++) zmax = fmaxf(zmax, z[e]);
-        for (uint32_t e = 0; e < a.NE; e++) zden += expf(z[e] - zmax);
+        for (uint32_t e = lane; e < a.NE; e += 32u) zmax = fmaxf(zmax, z[e]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) zmax = fmaxf(zmax, __shfl_xor_sync(0xffffffffu, zmax, o));
+        for (uint32_t e = lane; e < a.NE; e += 32u) zden += expf(z[e] - zmax);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) zden += __shfl_xor_sync(0xffffffffu, zden, o);
+    }
+    if (a.mode == 3u && a.keep < a.groups) {      // the experts of the groups that are not kept leave the choice
+        const uint32_t size = a.NE / a.groups;
+        for (uint32_t g = lane; g < a.groups; g += 32u) {
+            float b1 = -INFINITY, b2 = -INFINITY;
+            for (uint32_t e = g * size; e < (g + 1u) * size; e++) { const float v = z[e]; b2 = fmaxf(b2, fminf(b1, v)); b1 = fmaxf(b1, v); }
+            zg[g] = size > 1u ? b1 + b2 : b1;
+        }
+        __syncwarp();
+        for (uint32_t j = 0; j < a.keep; j++) {
+            float v;
+            const uint32_t g = warp_argmax(zg, a.groups, lane, &v);
+            __syncwarp();
+            if (lane == 0) zg[g] = -INFINITY;
+            __syncwarp();
+        }
+        for (uint32_t e = lane; e < a.NE; e += 32u) if (zg[e / size] != -INFINITY) z[e] = -INFINITY;
+        __syncwarp();
     }
     for (uint32_t j = 0; j < a.top; j++) {
-        float best = -INFINITY; uint32_t bi = 0xffffffffu;
-        for (uint32_t e = 0; e < a.NE; e++) {
-            const float v = z[e];
-            if (bi == 0xffffffffu || v > best) { best = v; bi = e; }
-        }
-        idx[j] = bi; wt[j] = best;
-        z[bi] = -INFINITY;                 // taken (a logit that IS -inf can only tie with taken ones after all finite ones are gone)
+        float best;
+        const uint32_t bi = warp_argmax(z, a.NE, lane, &best);
+        __syncwarp();
+        if (lane == 0) { idx[j] = bi; wt[j] = best; z[bi] = -INFINITY; }      // taken (a logit that IS -inf can only tie with taken ones after all finite ones are gone)
+        __syncwarp();
     }
+    if (lane) return;
     for (uint32_t k = 0; k < a.extra; k++) a.extra_out[(size_t)t * a.extra + k] = z[a.NE + k];
     if (a.mode == 1u) { for (uint32_t j = 0; j < a.top; j++) wt[j] = sigmoidf_(wt[j]); return; }
+    if (a.mode == 3u) { for (uint32_t j = 0; j < a.top; j++) wt[j] *= a.wscale; return; }
     if (a.mode == 2u) {      // the chosen experts' scores, divided by their sum
         float s = 0.0f;
         for (uint32_t j = 0; j < a.top; j++) { wt[j] = expf(wt[j] - zmax) / zden; s += wt[j]; }
@@ -1115,8 +1155,9 @@ __global__ void __launch_bounds__(256) k_route(const RouteArgs a) {
     extern __shared__ float z[];
     route_logits(a, blockIdx.x, z, z + a.NE + a.extra);
     __syncthreads();
+    if (threadIdx.x >= 32u) return;
+    route_pick(a, blockIdx.x, z, z + a.NE + a.extra);
     if (threadIdx.x) return;
-    route_pick(a, blockIdx.x, z);
     for (uint32_t j = 0; j < a.top; j++) atomicAdd(a.counts + a.idx[(size_t)blockIdx.x * a.top + j], 1u);
 }
 // Short portions: routing and placement of all T tokens in one block of 1024 threads (the one block has the router matrix to itself,
@@ -1128,7 +1169,7 @@ __global__ void __launch_bounds__(1024) k_route_small(const RouteArgs a) {
     for (uint32_t t = 0; t < a.T; t++) {
         route_logits(a, t, z, z + a.NE + a.extra);
         __syncthreads();
-        if (threadIdx.x == 0) route_pick(a, t, z);
+        if (threadIdx.x < 32u) route_pick(a, t, z, z + a.NE + a.extra);
         __syncthreads();
     }
     if (threadIdx.x) return;

@@ -253,9 +253,9 @@ __global__ void __launch_bounds__(256) k_retention_chain(const RetChainArgs a) {
     }
 }
 
-// each head's o divided by its root mean square over the value columns, times an optional gain (VD numbers, shared by the heads), times
+// each head's o divided by its root mean square over the value columns, times an optional gain (head h's VD numbers at h gain_stride; 0: shared), times
 // silu(gate), or sigmoid(gate) with sig: a warp per (token, head)
-struct RetOutArgs { const float *o; const float *g; uint32_t ldg; float *out; uint32_t T, H, VD; float eps; const float *gain; uint32_t sig; };
+struct RetOutArgs { const float *o; const float *g; uint32_t ldg; float *out; uint32_t T, H, VD; float eps; const float *gain; uint32_t sig; uint32_t gain_stride; };
 __global__ void __launch_bounds__(256) k_retention_out(const RetOutArgs a) {
     pdl_enter();
     const uint32_t warp = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31u;
@@ -267,7 +267,7 @@ __global__ void __launch_bounds__(256) k_retention_out(const RetOutArgs a) {
     s = warp_sum(s);
     const float rinv = 1.0f / sqrtf(s / (float)a.VD + a.eps);
     float *out = a.out + ((size_t)t * a.H + h) * a.VD;
-    for (uint32_t i = lane; i < a.VD; i += 32u) out[i] = o[i] * rinv * (a.gain ? a.gain[i] : 1.0f) * (a.sig ? sigmoidf_(g[i]) : siluf_(g[i]));
+    for (uint32_t i = lane; i < a.VD; i += 32u) out[i] = o[i] * rinv * (a.gain ? a.gain[h * a.gain_stride + i] : 1.0f) * (a.sig ? sigmoidf_(g[i]) : siluf_(g[i]));
 }
 
 // Window attention, first step.  One block per token, a warp per head: q (H heads) becomes unit-RMS times qmul[h] (the score scale

@@ -93,7 +93,8 @@ __global__ void __launch_bounds__(1024) k_post_norm(const PostNormArgs a) {
 
 // ------------------------------------------------------------------------------------------------
 // Grouped-query attention.  Rows of the joint product hold q [H][D] at q0, k [G][D] at k0, v [G][VD] at v0 and one gate number per head
-// at g0.  wq / wk (optional): gains of an RMS norm over ALL rows of q (of k) at once.  tab (optional): (cos, sin)[position][half];
+// at g0.  wq / wk (optional): gains of an RMS norm over ALL rows of q (of k) at once, or (head_norm) over every head by itself, D gains
+// shared by the heads.  block (0: none): a query sees the keys of its own block of that many positions only, counted from position 0.  tab (optional): (cos, sin)[position][half];
 // coordinate i < half turns with i + half, (u, v) -> (u cos - v sin, v cos + u sin); the rest of a head passes.  q carries the score
 // scale afterwards.  A cache row is [G D keys | G VD values | padding to 4].
 // ------------------------------------------------------------------------------------------------
@@ -102,7 +103,9 @@ struct GqaArgs {
     float *cache; const uint32_t *table; uint32_t T, H, G, D, VD, RL, pos0; const uint32_t *pos_ptr; float eps;
     float scale, softcap; const float *sink; uint32_t has_gate; float *out;      // softcap 0: none; sink null: none; out [T][H VD]
     uint32_t nsplit; float *part; uint32_t *tickets; uint32_t hb;                // k_gqa_decode: key splits; query heads per block
+    uint32_t block, head_norm;
 };
+__device__ __forceinline__ uint32_t gqa_first(uint32_t pos, uint32_t block) { return block ? pos - pos % block : 0u; }      // the first key position pos sees
 // coordinate d of one head: normed by r and its gains, turned
 __device__ __forceinline__ float rot_half_at(const float *x, const float *w, float r, uint32_t d, uint32_t half, const float2 *cs) {
     const float u = x[d] * r * (w ? w[d] : 1.0f);
@@ -119,7 +122,7 @@ __global__ void __launch_bounds__(256) k_qk_norm_rope(const GqaArgs a) {
     float *q = a.p + (size_t)t * a.ld + a.q0;
     const float *k = a.p + (size_t)t * a.ld + a.k0, *v = a.p + (size_t)t * a.ld + a.v0;
     float rq = 1.0f, rk = 1.0f;
-    if (a.wq || a.wk) {
+    if ((a.wq || a.wk) && !a.head_norm) {
         float2 s = make_float2(0.0f, 0.0f);
         for (uint32_t i = threadIdx.x; i < QW; i += blockDim.x) s.x = fmaf(q[i], q[i], s.x);
         for (uint32_t i = threadIdx.x; i < KW; i += blockDim.x) s.y = fmaf(k[i], k[i], s.y);
@@ -134,9 +137,14 @@ __global__ void __launch_bounds__(256) k_qk_norm_rope(const GqaArgs a) {
     for (uint32_t h = warp; h < a.H + a.G; h += nw) {
         const bool isq = h < a.H;
         const uint32_t hh = (isq ? h : h - a.H) * a.D;
-        const float *src = (isq ? q : k) + hh, *w = isq ? (a.wq ? a.wq + hh : nullptr) : (a.wk ? a.wk + hh : nullptr);
+        const float *src = (isq ? q : k) + hh, *w = isq ? a.wq : a.wk;
         float *dst = isq ? q + hh : row + hh;
-        const float r = isq ? rq * a.scale : rk;
+        float r = isq ? rq * a.scale : rk;
+        if (a.head_norm && w) {
+            float s = 0.0f;
+            for (uint32_t e = lane; e < a.D; e += 32u) s = fmaf(src[e], src[e], s);
+            r *= 1.0f / sqrtf(warp_sum(s) / (float)a.D + a.eps);
+        } else if (w) w += hh;
         for (uint32_t e = lane; e < per; e += 32u) {
             if (e < half) {
                 const float u = src[e] * r * (w ? w[e] : 1.0f), z = src[e + half] * r * (w ? w[e + half] : 1.0f);
@@ -171,7 +179,7 @@ __global__ void __launch_bounds__(256, VJ <= 2 ? 2 : 1) k_gqa_attn(const GqaArgs
     const uint32_t tid = threadIdx.x, ty = tid >> 4, tx = tid & 15u;
     const uint32_t r0 = (gridDim.x - 1u - blockIdx.x) * kGqaM;            // the longest tiles first
     const uint32_t pos = a.pos0 + (a.pos_ptr ? *a.pos_ptr : 0u);
-    const uint32_t t_last = (min(rows, r0 + kGqaM) - 1u) / rep, nkeys = pos + t_last + 1u, tiles = (nkeys + kGqaN - 1u) / kGqaN;
+    const uint32_t t_last = (min(rows, r0 + kGqaM) - 1u) / rep, nkeys = pos + t_last + 1u, tiles = (nkeys + kGqaN - 1u) / kGqaN, tile0 = gqa_first(pos + r0 / rep, a.block) / kGqaN;
     const bool vec = ((D | VD | a.ld | a.q0) & 3u) == 0;
     for (uint32_t i = tid; i < kGqaM * D4; i += 256u) {
         const uint32_t r = i / D4, d = (i % D4) * 4u, rr = r0 + r;
@@ -184,16 +192,16 @@ __global__ void __launch_bounds__(256, VJ <= 2 ? 2 : 1) k_gqa_attn(const GqaArgs
         *reinterpret_cast<float4 *>(q_s + r * LD + d) = v;
     }
     float m[4], l[4], o[4][VJ * 4];
-    uint32_t lim[4];                       // the last key each of this thread's rows sees
+    uint32_t lim[4], low[4];               // the last and the first key each of this thread's rows sees
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const uint32_t rr = min(r0 + ty * 4u + i, rows - 1u);
-        lim[i] = pos + rr / rep;
+        lim[i] = pos + rr / rep; low[i] = gqa_first(lim[i], a.block);
         m[i] = a.sink ? a.sink[g * rep + rr % rep] : -INFINITY; l[i] = a.sink ? 1.0f : 0.0f;
 #pragma unroll
         for (int c = 0; c < VJ * 4; c++) o[i][c] = 0.0f;
     }
-    for (uint32_t tile = 0; tile < tiles; tile++) {
+    for (uint32_t tile = tile0; tile < tiles; tile++) {
         __syncthreads();
         const uint32_t key0 = tile * kGqaN;
         // both pages of the tile; keys past the block's last one become zeros
@@ -238,7 +246,7 @@ __global__ void __launch_bounds__(256, VJ <= 2 ? 2 : 1) k_gqa_attn(const GqaArgs
             for (int j = 0; j < 4; j++) {
                 float v = s[i][j];
                 if (a.softcap > 0.0f) v = a.softcap * tanhf(v / a.softcap);
-                s[i][j] = key0 + tx + 16u * j <= lim[i] ? v : -INFINITY;
+                s[i][j] = key0 + tx + 16u * j <= lim[i] && key0 + tx + 16u * j >= low[i] ? v : -INFINITY;
                 tm = fmaxf(tm, s[i][j]);
             }
 #pragma unroll
@@ -310,10 +318,10 @@ __global__ void __launch_bounds__(256) k_gqa_decode(const GqaArgs a) {
     const uint32_t D = a.D, VD = a.VD, Dp = (D + 3u) & ~3u, VDp = (VD + 3u) & ~3u, rep = a.H / a.G, hgs = (rep + a.hb - 1u) / a.hb;
     const uint32_t g = blockIdx.y / hgs, h0 = g * rep + (blockIdx.y % hgs) * a.hb, nh = min(a.hb, (g + 1u) * rep - h0), t = blockIdx.z;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, key = tid >> 3, sub = tid & 7u;
-    const uint32_t pos = a.pos0 + (a.pos_ptr ? *a.pos_ptr : 0u), nkeys = pos + t + 1u, tiles = (nkeys + kPage - 1u) / kPage;
+    const uint32_t pos = a.pos0 + (a.pos_ptr ? *a.pos_ptr : 0u), nkeys = pos + t + 1u, low = gqa_first(pos + t, a.block), page0 = low / kPage, tiles = (nkeys + kPage - 1u) / kPage - page0;
     const uint32_t tps = (tiles + a.nsplit - 1u) / a.nsplit, nact = (tiles + tps - 1u) / tps, split = blockIdx.x;
     if (split >= nact) return;
-    const uint32_t tile_lo = split * tps, tile_hi = min(tiles, tile_lo + tps), half = a.tab ? a.half : 0u;
+    const uint32_t tile_lo = page0 + split * tps, tile_hi = min(page0 + tiles, tile_lo + tps), half = a.tab ? a.half : 0u;
     float *q_s = sm;                                   // [kGqaHeads][Dp]
     float *kn_s = q_s + kGqaHeads * Dp;                // [kGemvMaxM][Dp]: the portion's own keys
     float *v_s = kn_s + kGemvMaxM * Dp;                // [kPage][VDp]
@@ -346,32 +354,38 @@ __global__ void __launch_bounds__(256) k_gqa_decode(const GqaArgs a) {
     };
     fetch(tile_lo);
     // Norm factors are numbers per token: queries and keys are gained and turned without them (no wait for the sums), the scores and the
-    // cached key carry them.  red[0]: the whole query row's sum of squares; red[1 + u]: the key row's of the portion's token u (tail shares)
+    // cached key carry them.  red[0]: the whole query row's sum of squares; red[1 + u]: the key row's of the portion's token u (tail shares).
+    // Norms per head: red[0][h] is head h's own sum, and one warp makes the whole of red[1 + u].
     const uint32_t QW = a.H * D, KW = a.G * D;
     {
         float s[1 + kGemvMaxM];
 #pragma unroll
         for (uint32_t u = 0; u <= kGemvMaxM; u++) s[u] = 0.0f;
-        if (a.wq) {
+        if (a.head_norm) {
+            if (a.wq && warp < nh) { const float *q = a.p + (size_t)t * a.ld + a.q0 + (h0 + warp) * D; for (uint32_t i = lane; i < D; i += 32u) s[0] = fmaf(q[i], q[i], s[0]); }
+#pragma unroll
+            for (uint32_t u = 0; u < kGemvMaxM; u++)
+                if (a.wk && tail && u == warp && u <= t) { const float *k = a.p + (size_t)u * a.ld + a.k0 + g * D; for (uint32_t i = lane; i < D; i += 32u) s[1 + u] = fmaf(k[i], k[i], s[1 + u]); }
+        } else if (a.wq) {
             const float *q = a.p + (size_t)t * a.ld + a.q0;
             if (VEC) {
 #pragma unroll 4
                 for (uint32_t i = tid; i < QW / 4u; i += 256u) { const float4 v = reinterpret_cast<const float4 *>(q)[i]; s[0] = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s[0])))); }
             } else for (uint32_t i = tid; i < QW; i += 256u) s[0] = fmaf(q[i], q[i], s[0]);
         }
-        if (a.wk && tail) {
+        if (a.wk && tail && !a.head_norm) {
 #pragma unroll
             for (uint32_t u = 0; u < kGemvMaxM; u++)
                 if (u <= t) { const float *k = a.p + (size_t)u * a.ld + a.k0; for (uint32_t i = tid; i < KW; i += 256u) s[1 + u] = fmaf(k[i], k[i], s[1 + u]); }
         }
         for (uint32_t i = tid; i < nh * Dp; i += 256u) {
             const uint32_t h = i / Dp, d = i % Dp;
-            q_s[i] = d < D ? rot_half_at(a.p + (size_t)t * a.ld + a.q0 + (h0 + h) * D, a.wq ? a.wq + (h0 + h) * D : nullptr, 1.0f, d, half, a.tab + (size_t)(pos + t) * half) : 0.0f;
+            q_s[i] = d < D ? rot_half_at(a.p + (size_t)t * a.ld + a.q0 + (h0 + h) * D, a.wq ? a.wq + (a.head_norm ? 0u : (h0 + h) * D) : nullptr, 1.0f, d, half, a.tab + (size_t)(pos + t) * half) : 0.0f;
         }
         if (tail)
             for (uint32_t i = tid; i < (t + 1u) * Dp; i += 256u) {
                 const uint32_t u = i / Dp, d = i % Dp;
-                kn_s[i] = d < D ? rot_half_at(a.p + (size_t)u * a.ld + a.k0 + g * D, a.wk ? a.wk + g * D : nullptr, 1.0f, d, half, a.tab + (size_t)(pos + u) * half) : 0.0f;
+                kn_s[i] = d < D ? rot_half_at(a.p + (size_t)u * a.ld + a.k0 + g * D, a.wk ? a.wk + (a.head_norm ? 0u : g * D) : nullptr, 1.0f, d, half, a.tab + (size_t)(pos + u) * half) : 0.0f;
             }
 #pragma unroll
         for (uint32_t u = 0; u <= kGemvMaxM; u++) { s[u] = warp_sum(s[u]); if (lane == 0) red[u][warp] = s[u]; }
@@ -384,10 +398,11 @@ __global__ void __launch_bounds__(256) k_gqa_decode(const GqaArgs a) {
         for (uint32_t w = 0; w < 8u; w++) v += red[j][w];
         return 1.0f / sqrtf(v / (float)n + a.eps);
     };
-    const float qf = factor(0, a.wq != nullptr, QW) * a.scale;
+    const uint32_t QN = a.head_norm ? D : QW, KN = a.head_norm ? D : KW;
+    const float qf = (a.head_norm && a.wq ? 1.0f / sqrtf(red[0][sub] / (float)QN + a.eps) : factor(0, a.wq != nullptr, QN)) * a.scale;      // of head `sub`, or of all
     if (split == nact - 1u && blockIdx.y % hgs == 0) {            // one block writes the token's row of this key/value head
         float *row = a.cache + ((size_t)a.table[(pos + t) / kPage] * kPage + (pos + t) % kPage) * a.RL;
-        const float kf = factor(1u + t, a.wk != nullptr, KW);
+        const float kf = factor(1u + t, a.wk != nullptr, KN);
         for (uint32_t d = tid; d < D; d += 256u) row[g * D + d] = kn_s[t * Dp + d] * kf;
         for (uint32_t d = tid; d < VD; d += 256u) row[a.G * D + g * VD + d] = a.p[(size_t)t * a.ld + a.v0 + g * VD + d];
     }
@@ -397,7 +412,7 @@ __global__ void __launch_bounds__(256) k_gqa_decode(const GqaArgs a) {
     for (uint32_t tile = tile_lo; tile < tile_hi; tile++) {
         const uint32_t kp = tile * kPage + key;
         if (kp >= pos && kp < nkeys) {
-            const float kf = factor(1u + kp - pos, a.wk != nullptr, KW);
+            const float kf = factor(1u + kp - pos, a.wk != nullptr, KN);
 #pragma unroll
             for (int c = 0; c < CH; c++) {
                 const uint32_t d = (sub + 8u * c) * 4u;
@@ -429,7 +444,7 @@ __global__ void __launch_bounds__(256) k_gqa_decode(const GqaArgs a) {
         if (warp < nh) {
             float s = s_s[warp * kPage + lane];
             if (a.softcap > 0.0f) s = a.softcap * tanhf(s / a.softcap);
-            const bool seen = tile * kPage + lane < nkeys;
+            const bool seen = tile * kPage + lane < nkeys && tile * kPage + lane >= low;
             s = seen ? s : -INFINITY;
             float tm = s;
 #pragma unroll

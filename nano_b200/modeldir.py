@@ -1,5 +1,5 @@
-"""Model folders (config.json + model.safetensors) from the Python side: a writer, and random-weight Famudra, Rakarax, Gokinex, Vumunex and
-Kadesun models for the benchmarks and tests.  The reader the engine uses is native (csrc/modeldir.cu); nothing here is on the compute path.
+"""Model folders (config.json + model.safetensors) from the Python side: a writer, and random-weight Famudra, Rakarax, Gokinex, Vumunex,
+Kadesun and Fidatar models for the benchmarks and tests.  The reader the engine uses is native (csrc/modeldir.cu); nothing here is on the compute path.
 
 A safetensors file is an 8-byte little-endian header length, that many bytes of JSON (name -> dtype, shape, data_offsets) and
 the tensor bytes.
@@ -373,4 +373,58 @@ def kadesun_random(config: dict, seed: int = 0, gain: float = 1.0, decay_rank: i
         if f:
             t[p + "norm2"] = vecn(E, 0.4, 0.9)
             t[p + "mlp.gate"] = lin(f["ff"], E, 1.5); t[p + "mlp.up"] = lin(f["ff"], E); t[p + "mlp.down"] = lin(E, f["ff"])
+    return t
+
+
+def fidatar_config(vocab: int, width: int, layers, alpha: float = 1.5, scale: float = 4.0, softcap=20.0, eps: float = 1e-5) -> dict:
+    """layers: list of (type, mixer, mlp).
+    type "attention": mixer {heads, kv_heads, dim, vdim, scale, mask: {size} (optional), rot: {dims, base, scaling: {factor, original,
+    fast, slow} (optional)} (optional)}; type "mlstm": mixer {heads, dim, vdim, gate_cap}; mlp: None, {"kind": "dense", "ff": f} or
+    {"kind": "moe", "router": {"experts": n, "top": k, "groups": {"count": c, "keep": k}, "scale": s}, "expert": {"ff": f}}.
+    alpha: the residual's factor before the norms of the sums; scale: of the embedding; softcap: of the logits (None: the key is left out)."""
+    out = [{"type": kind, "mixer": json.loads(json.dumps(mixer)), "mlp": json.loads(json.dumps(mlp)) if mlp else None} for kind, mixer, mlp in layers]
+    cfg = {"architecture": "Fidatar", "vocab": vocab, "width": width, "embedding": {"scale": scale}, "norm": {"eps": eps}, "postln_alpha": alpha, "layers": out}
+    if softcap is not None:
+        cfg["logit_softcap"] = softcap
+    return cfg
+
+
+def fidatar_random(config: dict, seed: int = 0, gain: float = 1.0) -> Dict[str, np.ndarray]:
+    """Random weights (bfloat16-representable fp32 arrays) for a Fidatar config: projections ~ N(0, gain^2 / fan_in)."""
+    rng = np.random.default_rng(seed)
+    E, V = config["width"], config["vocab"]
+
+    def lin(o, i, g=1.0):
+        return bf16_round((rng.standard_normal((o, i), dtype=np.float32) * (gain * g / np.sqrt(i))).astype(np.float32))
+
+    def vecn(n, lo, hi):
+        return bf16_round(rng.uniform(lo, hi, size=n).astype(np.float32))
+
+    t = {"embed": bf16_round(rng.standard_normal((V, E), dtype=np.float32) / np.float32(config["embedding"]["scale"])), "head": lin(V, E, 4.0), "final.norm": vecn(E, 0.7, 1.3)}
+    for i, L in enumerate(config["layers"]):
+        p = f"l{i}."
+        t[p + "norm1"] = vecn(E, 0.7, 1.3)
+        m = L["mixer"]
+        q = p + "mix."
+        H, D, VD = m["heads"], m["dim"], m["vdim"]
+        if L["type"] == "attention":
+            G = m["kv_heads"]
+            for n, rows in (("q", H * D), ("k", G * D), ("v", G * VD)):
+                t[q + n] = lin(rows, E); t[q + n + ".b"] = vecn(rows, -0.5, 0.5)
+            t[q + "q.norm"] = vecn(D, 0.7, 1.6); t[q + "k.norm"] = vecn(D, 0.7, 1.6)
+            t[q + "o"] = lin(E, H * VD, 2.0)
+        else:
+            t[q + "q"] = lin(H * D, E, 1.5); t[q + "k"] = lin(H * D, E, 1.5); t[q + "v"] = lin(H * VD, E, 1.5); t[q + "g"] = lin(H * VD, E, 1.5)
+            t[q + "i"] = lin(H, E, 2.0); t[q + "i.b"] = vecn(H, -2.0, 1.0); t[q + "f"] = lin(H, E, 1.5); t[q + "f.b"] = vecn(H, 1.0, 5.0)
+            t[q + "norm"] = vecn(H * VD, 0.6, 1.4); t[q + "o"] = lin(E, H * VD, 2.0)
+        f = L.get("mlp")
+        if not f:
+            continue
+        t[p + "norm2"] = vecn(E, 0.7, 1.3)
+        if f["kind"] == "dense":
+            t[p + "mlp.up"] = lin(f["ff"], E, 1.2); t[p + "mlp.down"] = lin(E, f["ff"])
+        else:
+            t[p + "mlp.router"] = lin(f["router"]["experts"], E, 2.0)
+            for e in range(f["router"]["experts"]):
+                t[p + f"mlp.e{e}.up"] = lin(f["expert"]["ff"], E, 1.2); t[p + f"mlp.e{e}.down"] = lin(E, f["expert"]["ff"])
     return t
