@@ -933,6 +933,89 @@ def kadesun_bench(args):
                       "clocks": clocks, "sizes": out}))
 
 
+# --------------------------------------------------------------------------------------------------
+# --design fidatar: the same two measurements for the Fidatar design (grouped-query attention in blocks of positions, matrix memory with
+# exponential gates, squared-relu dense and routed feed-forwards, norms of the residual sums) beside the closest model of the same runtime,
+# Kadesun (grouped-query attention beside and between matrix states of the same size, dense feed-forwards), at equal width and depth.
+# --------------------------------------------------------------------------------------------------
+FIDATAR_SIZES = {
+    # name: (width, layers, attention heads, kv heads, dim, vdim, memory heads, dim, vdim, dense ff, experts, top, groups, kept, expert ff)
+    "w1024": (1024, 8, 16, 4, 64, 64, 8, 128, 128, 4096, 16, 2, 4, 2, 1024),
+    "w2048": (2048, 8, 16, 4, 128, 128, 16, 128, 128, 8192, 16, 2, 4, 2, 2048),
+}
+
+
+def fidatar_model(name):
+    from nano_b200 import modeldir as md
+    E_, L, H, G, D, VD, MH, MD, MVD, ff, NE, top, count, kept, eff = FIDATAR_SIZES[name]
+    att = {"heads": H, "kv_heads": G, "dim": D, "vdim": VD, "scale": D ** -0.5, "mask": {"size": 4096},
+           "rot": {"dims": D // 2, "base": 10000.0, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+    mem = {"heads": MH, "dim": MD, "vdim": MVD, "gate_cap": 15.0}
+    moe = {"kind": "moe", "router": {"experts": NE, "top": top, "groups": {"count": count, "keep": kept}, "scale": 1.5}, "expert": {"ff": eff}}
+    layers = [("attention", att, {"kind": "dense", "ff": ff}) if i % 2 == 0 else ("mlstm", mem, moe) for i in range(L)]
+    cfg = md.fidatar_config(FAMUDRA_VOCAB, E_, layers, alpha=2.5, scale=E_ ** 0.5, softcap=30.0)
+    path = os.path.join(os.environ.get("NB200_MODEL_CACHE", "/tmp/nb200_models"), f"fidatar-{name}")
+    if not os.path.exists(os.path.join(path, "model.safetensors")):
+        md.write_model_dir(path + ".part", cfg, md.fidatar_random(cfg, 0))
+        os.replace(path + ".part", path)
+    return path, cfg
+
+
+def fidatar_decode_bytes(cfg, pos, wbytes=2):
+    """Algorithmic HBM bytes of one decoded token at position pos: every matrix once (top-k experts only), the fp32 states read and
+    written, the fp32 key and value rows of every earlier position (all of them in one block here), the head."""
+    E_ = cfg["width"]; b = 0.0
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        H, D, VD = m["heads"], m["dim"], m["vdim"]
+        if L["type"] == "attention":
+            b += wbytes * (H * (D + VD) + m["kv_heads"] * (D + VD)) * E_ + 4.0 * m["kv_heads"] * (D + VD) * (pos + 1)
+        else:
+            b += wbytes * (2 * H * D + 3 * H * VD + 2 * H) * E_ + 8.0 * H * (D * VD + D)
+        f = L["mlp"]
+        if f["kind"] == "dense":
+            b += wbytes * 2 * E_ * f["ff"]
+        else:
+            b += 4.0 * f["router"]["experts"] * E_ + wbytes * 2 * E_ * f["router"]["top"] * f["expert"]["ff"]
+    return b + wbytes * cfg["vocab"] * E_
+
+
+def fidatar_flops_per_token(cfg, ctx):
+    fl = 2.0 * (fidatar_decode_bytes(cfg, 0, 1) - cfg["vocab"] * cfg["width"])
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        H, D, VD = m["heads"], m["dim"], m["vdim"]
+        if L["type"] == "attention":
+            fl += 2.0 * H * (D + VD) * ctx
+        else:
+            fl += H * (4.0 * D * VD + 2.0 * 32.5 * (D + VD)) - 16.0 * H * (D * VD + D)          # k v^T and q S, the causal products of 64-token chunks; the state's bytes are no products
+    return fl
+
+
+def fidatar_bench(args):
+    from nano_b200 import engine as E
+    hbm, hbm_src = peaks()
+    try:
+        tf = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    except Exception:
+        tf = 1590.0
+    ctx, n_dec, T = 1024, 128, 2048
+    sampler = ClockSampler(0); sampler.start()
+    out = {}
+    for name in (args.sizes.split(",") if args.sizes else sorted(FIDATAR_SIZES)):
+        path, cfg = fidatar_model(name)
+        row = layered_modes(E, path, FAMUDRA_VOCAB, ctx, n_dec, T, args, hbm, tf, lambda pos, wb: fidatar_decode_bytes(cfg, pos, wb), lambda c: fidatar_flops_per_token(cfg, c))
+        ppath, pcfg = kadesun_model(name)          # the closest model: the same runtime's Kadesun at equal width and depth
+        args_bf16 = argparse.Namespace(**{**vars(args), "with_f32": False})
+        row["peer_kadesun"] = layered_modes(E, ppath, FAMUDRA_VOCAB, ctx, n_dec, T, args_bf16, hbm, tf, lambda pos, wb: kadesun_decode_bytes(pcfg, pos, wb), lambda c: kadesun_flops_per_token(pcfg, c))["bf16"]
+        out[name] = row
+    clocks = sampler.stop()
+    print(json.dumps({"design": "fidatar", "unit": "tokens/s", "n_gpus": 1, "data": "synthetic (random weights)", "peaks": {"hbm_gbs": hbm, "hbm_source": hbm_src, "bf16_tflops": tf},
+                      "config": {"decode": f"greedy device loop, {n_dec} tokens after a {ctx}-token prompt, batch 1", "prefill": f"one portion of {T} tokens into an empty sequence",
+                                 "timing": "CUDA events on the engine's stream after warm-up", "l2": "fractions are against HBM although the weights of one token fit the 126 MB L2 at w1024"},
+                      "clocks": clocks, "sizes": out}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -949,7 +1032,7 @@ def main():
     ap.add_argument("--no-pdl", action="store_true")
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--no-stream", action="store_true", help="forbid the streaming kernel")
-    ap.add_argument("--design", default=None, choices=["famudra", "rakarax", "gokinex", "vumunex", "kadesun"], help="measure a model-folder design instead of the headline workload (its own JSON line)")
+    ap.add_argument("--design", default=None, choices=["famudra", "rakarax", "gokinex", "vumunex", "kadesun", "fidatar"], help="measure a model-folder design instead of the headline workload (its own JSON line)")
     ap.add_argument("--sizes", default=None, help="--design: comma-separated size names (default: all)")
     ap.add_argument("--with-f32", action="store_true", help="--design: also time the true-32-bit mode")
     args = ap.parse_args()
@@ -967,6 +1050,9 @@ def main():
         return
     if args.design == "kadesun":
         kadesun_bench(args)
+        return
+    if args.design == "fidatar":
+        fidatar_bench(args)
         return
     args.warmup = max(args.warmup, 3) if args.impl == "b200" else args.warmup
 

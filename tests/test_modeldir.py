@@ -216,3 +216,71 @@ def test_kadesun_oracle_is_causal_and_follows_the_delta_rule():
     d = O.delta_rule(KAD_DELTA, tt, "l1.mix.", res[0], 1e-5)
     assert np.allclose(res[1], res[0] + O.rms_norm(d, tt["l1.norm1"], 1e-5), atol=1e-12)
 
+
+
+FID_ATT = {"heads": 4, "kv_heads": 2, "dim": 8, "vdim": 6, "scale": 0.4, "mask": {"size": 5}, "rot": {"dims": 4, "base": 100.0, "scaling": {"factor": 4.0, "original": 30, "fast": 4.0, "slow": 0.5}}}
+FID_MEM = {"heads": 2, "dim": 6, "vdim": 10, "gate_cap": 8.0}
+FID_MOE = {"kind": "moe", "router": {"experts": 6, "top": 2, "groups": {"count": 3, "keep": 2}, "scale": 1.5}, "expert": {"ff": 7}}
+
+
+@pytest.mark.skipif(E.device_count() > 0, reason="box has a GPU")
+def test_fidatar_folder_reaches_the_layered_family(tmp_path):
+    cfg = md.fidatar_config(16, 8, [("attention", FID_ATT, {"kind": "dense", "ff": 12}), ("mlstm", FID_MEM, FID_MOE), ("mlstm", FID_MEM, None)])
+    w = md.fidatar_random(cfg)
+    assert w["l0.mix.q.norm"].shape == (8,) and w["l1.mix.norm"].shape == (20,) and w["l1.mlp.e5.down"].shape == (8, 7) and "l2.norm2" not in w
+    p = md.write_model_dir(str(tmp_path / "f"), cfg, w)
+    with pytest.raises(E.NB200Error, match="no CUDA device"):
+        E.Engine(p, 16)
+
+
+def test_fidatar_oracle_is_causal_and_follows_its_parts():
+    """The plain restatement itself: a prefix gives the same logits; attention stays inside its block and turns by relative positions; the
+    one takes weight away; the memory equals its unstabilised sums whatever the running maximum, and a state carried over equals one pass;
+    groups; the rescaled rotation keeps fast pairs, divides slow ones and blends between; the residual is normed after every sum."""
+    import fidatar_oracle as O
+    rng = np.random.default_rng(0)
+    cfg = md.fidatar_config(20, 16, [("attention", FID_ATT, {"kind": "dense", "ff": 12}), ("mlstm", FID_MEM, FID_MOE)])
+    w = md.fidatar_random(cfg, 3)
+    t = rng.integers(0, 20, 24)
+    full = O.forward(cfg, w, t)
+    assert np.allclose(O.forward(cfg, w, t[:10]), full[:10], atol=1e-12) and np.abs(full).max() < 20.0
+    tt = {n: np.asarray(x, np.float64) for n, x in w.items()}
+    h = rng.standard_normal((24, 16))
+    y = O.attention(FID_ATT, tt, "l0.mix.", h, 1e-5)
+    h2 = h.copy(); h2[:10] = rng.standard_normal((10, 16))
+    assert np.allclose(O.attention(FID_ATT, tt, "l0.mix.", h2, 1e-5)[10:], y[10:], atol=1e-12)
+    h3 = np.concatenate([h[5:10], h[5:10]])
+    y3 = O.attention(FID_ATT, tt, "l0.mix.", h3, 1e-5)
+    assert np.allclose(y3[:5], y3[5:], atol=1e-12)
+    one = O.attention(FID_ATT, tt, "l0.mix.", h[:1], 1e-5)[0]
+    k = O.rms_norm((h[0] @ tt["l0.mix.k"].T + tt["l0.mix.k.b"]).reshape(2, 8), tt["l0.mix.k.norm"], 1e-5)
+    q = O.rms_norm((h[0] @ tt["l0.mix.q"].T + tt["l0.mix.q.b"]).reshape(4, 8), tt["l0.mix.q.norm"], 1e-5)
+    amp = (0.1 * np.log(4.0) + 1.0) * np.array([1, 1, 1, 1, 0, 0, 0, 0]) + np.array([0, 0, 0, 0, 1, 1, 1, 1])
+    v = (h[0] @ tt["l0.mix.v"].T + tt["l0.mix.v.b"]).reshape(2, 6)
+    s = np.exp(0.4 * np.array([(q[a] * amp) @ (k[a // 2] * amp) for a in range(4)]))
+    assert np.allclose(one, np.concatenate([s[a] / (1 + s[a]) * v[a // 2] for a in range(4)]) @ tt["l0.mix.o"].T)
+    f, a = O.rotation_frequencies({"dims": 16, "base": 1000.0, "scaling": {"factor": 8.0, "original": 400, "fast": 16.0, "slow": 0.5}})
+    raw = 1000.0 ** (-np.arange(8) / 8.0)
+    assert np.allclose(f[0], raw[0]) and np.allclose(f[-1] / raw[-1], 1.0 / 8.0) and (np.diff(f / raw) <= 1e-15).all() and np.isclose(a, 1 + 0.1 * np.log(8.0))
+    q, k, v = rng.standard_normal((6, 2, 5)), rng.standard_normal((6, 2, 5)), rng.standard_normal((6, 2, 3))
+    li, lf = rng.uniform(-3, 3, (6, 2)), O.log_sigmoid(rng.uniform(-2, 4, (6, 2)))
+    o, S = O.memory(q, k, v, li, lf)
+    for head in range(2):
+        for i in range(6):
+            g = np.array([np.exp(lf[j + 1:i + 1, head].sum() + li[j, head]) for j in range(i + 1)])
+            num = (g * (k[:i + 1, head] @ q[i, head])) @ v[:i + 1, head]
+            den = max(abs((g * (k[:i + 1, head] @ q[i, head])).sum()), 1.0)
+            assert np.allclose(o[i, head], num / den, rtol=1e-4)
+    o1, S1 = O.memory(q[:4], k[:4], v[:4], li[:4], lf[:4])
+    o2, S2 = O.memory(q[4:], k[4:], v[4:], li[4:], lf[4:], S1)
+    assert np.allclose(np.concatenate([o1, o2]), o) and all(np.allclose(x, z) for x, z in zip(S2, S))
+    z = np.array([[2.0, -3.0, 1.0, 0.9, -1.0, 1.9]])
+    idx, wt = O.router(FID_MOE, {"r.router": np.eye(6)}, "r.", z)
+    assert list(idx[0]) == [5, 2]          # the pair (1, 0.9) outweighs the pair (2, -3)
+    assert np.allclose(wt[0, 0], 1.5 * O.sigmoid(z[0, idx[0, 0]]))
+    res = []
+    O.forward(cfg, w, t, res)
+    x = tt["embed"][t] * 4.0
+    x = O.rms_norm(1.5 * x + O.attention(FID_ATT, tt, "l0.mix.", x, 1e-5), tt["l0.norm1"], 1e-5)
+    x = O.rms_norm(1.5 * x + O.dense_ff(tt, "l0.mlp.", x), tt["l0.norm2"], 1e-5)
+    assert np.allclose(res[0], x, atol=1e-12)
