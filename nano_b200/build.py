@@ -57,8 +57,7 @@ def build_engine(force: bool = False, verbose: bool = False, units=None, target:
     units / target: a library of a subset of the families (build_layered)."""
     os.makedirs(LIB, exist_ok=True)
     target = target or ENGINE_SO
-    base = [NVCC, "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC",
-            "--split-compile", "0"]          # the kernels of one unit are optimised side by side
+    base = [NVCC, "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC"]
     if verbose:
         base.insert(1, "-Xptxas=-v")
     objs, procs = [], []

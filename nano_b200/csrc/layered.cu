@@ -185,7 +185,7 @@ struct LayeredEngine : nb::EngineBase {
     float *b_wpart = nullptr, *b_rseg = nullptr; uint32_t *b_wtick = nullptr, *b_rtick = nullptr;      // window attention: partials and tickets of the key splits
     float *b_p = nullptr, *b_qk = nullptr, *b_xc = nullptr, *b_a = nullptr, *b_ro = nullptr, *b_dbc = nullptr, *b_dt = nullptr, *b_y = nullptr, *b_f = nullptr;   // retention, window attention + selective scan, dense feed-forward
     uint32_t *b_tick = nullptr;      // attention: tickets of the key splits
-    uint32_t *b_idx = nullptr, *b_cnt = nullptr, *b_off = nullptr, *b_fill = nullptr, *b_slot = nullptr, *b_rows = nullptr;
+    uint32_t *b_idx = nullptr, *b_cnt = nullptr, *b_off = nullptr, *b_fill = nullptr, *b_act = nullptr, *b_slot = nullptr, *b_rows = nullptr;
     float *b_xn = nullptr, *logits = nullptr, *keep = nullptr;
     // Dynamic-Tanh designs: embedding scale, the pair table and its hash, the norms around the stack, where a slot keeps the last token
     int norm_kind = NORM_RMS_ZERO; float emb_scale = 1.0f; Weight pairs; uint32_t buckets = 0, mul_prev = 0, mul_cur = 0; Dyt embed_norm{}, final_dyt{}; size_t st_tok = 0;
@@ -889,6 +889,7 @@ int gemm(LayeredEngine *e, GemmArgs a, uint32_t groups, uint32_t maxM, bool wf32
     if (maxM <= kGemvMaxM) {
         a.round_a = f32 ? 0u : 1u;
         const uint32_t gx = gemv_blocks(e, a.N, active ? std::min(active, groups) : groups);
+        if (a.g_act && active) groups = std::min(active, groups);          // only the groups with rows are launched
         if (a.epi == EPI_CONV_RANGES)
             return f32 ? launch<GemmArgs>(e, k_gemv_ext<float, 1>, dim3(gx, groups), dim3(256), 0, a) : launch<GemmArgs>(e, k_gemv_ext<__nv_bfloat16, 1>, dim3(gx, groups), dim3(256), 0, a);
         if (a.res_x && a.a_parts <= 1)
@@ -1393,8 +1394,8 @@ int mix_gqa(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) {
 }
 
 // ---- matrix memory ----
-// one product gives [q | k | v | g | i | f]; short portions: the rest up to the output product is one kernel; long ones: gates, states
-// before every chunk, outputs of all chunks, norm and gate
+// one product gives [q | k | v | g | i | f]; short portions: the rest up to the output product is one kernel; long ones: gates, what
+// every chunk writes, the states before them, outputs of all chunks, norm and gate
 int mix_memory(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) {
     const uint32_t T = cx.T, H = L.H, D = L.dim, VD = L.vdim, P = L.proj.rows, k0 = H * D, v0 = 2 * H * D, g0 = v0 + H * VD, i0 = L.c_if, f0 = i0 + H;
     const float qscale = (float)(1.0 / sqrt((double)D));
@@ -1415,10 +1416,12 @@ int mix_memory(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) 
     }
     const uint32_t chunks = (T + kMemChunk - 1u) / kMemChunk;
     MemGatesArgs ga{e->b_p, P, i0, f0, L.gate_cap, m, e->b_mfa, e->b_mfb, e->b_mfc, e->b_mmt, e->b_mme, T, H, chunks};
-    MemStatesArgs sa{e->b_p, P, k0, v0, e->b_mfb, e->b_mfc, e->b_mme, S, n, e->b_mS, e->b_mn, T, H, D, VD, chunks};
+    MemWriteArgs wa{e->b_p, P, k0, v0, e->b_mfb, e->b_mfc, e->b_mme, e->b_mS, e->b_mn, T, H, D, VD, chunks};
+    MemChainArgs ca{e->b_mfc, e->b_mme, S, n, e->b_mS, e->b_mn, H, D, VD, chunks};
     MemOutArgs oa{e->b_p, P, 0u, k0, v0, qscale, e->b_mfa, e->b_mfb, e->b_mmt, e->b_mme, e->b_mS, e->b_mn, e->b_mo, T, H, D, VD, chunks};
     if ((r = launch<MemGatesArgs>(e, k_memory_gates, dim3(H), dim3(1024), 0, ga)) ||
-        (r = launch<MemStatesArgs>(e, k_memory_states, dim3((VD + 31u) / 32u, (D + 63u) / 64u, H), dim3(256), 0, sa))) return r;
+        (r = launch<MemWriteArgs>(e, k_memory_writes, dim3((VD + 63u) / 64u, (D + 63u) / 64u, chunks * H), dim3(256), 0, wa)) ||
+        (r = launch<MemChainArgs>(e, k_memory_chain, dim3((VD * D + D + 255u) / 256u, H), dim3(256), 0, ca))) return r;
     // 128 value columns per block (the scores are made once for them) where that still fills the GPU twice
     if (VD > 64u && (VD + 127u) / 128u * chunks * H >= 2u * (uint32_t)e->num_sms) r = launch<MemOutArgs>(e, k_memory_out<2>, dim3((VD + 127u) / 128u, chunks, H), dim3(256), memory_out_smem(2), oa);
     else r = launch<MemOutArgs>(e, k_memory_out<1>, dim3((VD + 63u) / 64u, chunks, H), dim3(256), memory_out_smem(1), oa);
@@ -1472,6 +1475,12 @@ int ff_glu_dense(LayeredEngine *e, const Layer &L, uint32_t T) {
     return last_product(e, plain(e->b_f2, L.ff, L.down, e->d, e->E, T), T);
 }
 
+// routing of a short portion: a cluster of blocks shares the router's rows
+int route_small(LayeredEngine *e, const RouteArgs &ra) {
+    const uint32_t NL = ra.NE + ra.extra, nb = NL >= 8u ? kRouteBlocks : NL >= 4u ? 4u : NL >= 2u ? 2u : 1u;
+    return launch<RouteArgs>(e, k_route_small, dim3(nb), dim3(kRouteThreads), route_small_smem(NL), ra, nb);
+}
+
 // experts chosen by sigmoid scores: e->h2 -> the rows of e->b_eo (one per token and choice, in expert order) and, with a shared expert,
 // e->b_so and the gate logits e->b_sg; the residual kernel adds them up.  The score weights the expert's INPUT; the experts have no
 // bias, so act(s g) (s u) of the unweighted products g, u is the same number.  The shared expert runs on a second stream.
@@ -1482,11 +1491,11 @@ int ff_moe_scored(LayeredEngine *e, const Layer &L, uint32_t T) {
     if (L.has_shared && e->branch_streams) CK(cudaEventRecord(e->ev_fork, e->stream));
     float *wrow = L.score_in ? e->b_wrow : nullptr;
     RouteArgs ra{e->h2, L.router, e->b_idx, e->b_wt, e->b_cnt, e->b_off, e->b_fill, e->b_slot, e->b_rows, T, L.NE, L.top, E, L.route_mode, L.sh_gate ? 1u : 0u, e->b_sg, wrow};
-    if (small) { if ((r = launch<RouteArgs>(e, k_route_small, dim3(1), dim3(1024), route_smem(NL, 1024), ra))) return r; }
+    if (small) { ra.act = e->b_act; if ((r = route_small(e, ra))) return r; }
     else if ((r = launch<RouteArgs>(e, k_route, dim3(T), dim3(256), route_smem(NL, 256), ra)) || (r = launch<RouteArgs>(e, k_route_place, dim3(1), dim3(1024), 0, ra))) return r;
     GemmArgs u{};
     u.A = e->h2; u.lda = E; u.W = L.up.p; u.ldw = E; u.M = T; u.K = E; u.a_gmod = 1;
-    u.g_off = e->b_off; u.a_rows = e->b_rows; u.w_gstride = (uint64_t)2 * L.ff * E;
+    u.g_off = e->b_off; u.a_rows = e->b_rows; u.g_act = small ? e->b_act : nullptr; u.w_gstride = (uint64_t)2 * L.ff * E;
     if (small) { u.C = e->b_hb; u.ldc = L.ff; u.N = L.ff; u.glu = L.glu_kind; u.glu_limit = L.limit; u.row_scale = wrow; }
     else { u.C = e->b_hg; u.ldc = 2 * L.ff; u.N = 2 * L.ff; }
     if ((r = gemm(e, u, L.NE, T, false, T * L.top))) return r;
@@ -1496,7 +1505,7 @@ int ff_moe_scored(LayeredEngine *e, const Layer &L, uint32_t T) {
     }
     GemmArgs dn{};
     dn.A = e->b_hb; dn.lda = L.ff; dn.W = L.down.p; dn.ldw = L.ff; dn.C = e->b_eo; dn.ldc = E; dn.M = T; dn.N = E; dn.K = L.ff; dn.a_gmod = 1;
-    dn.g_off = e->b_off; dn.w_gstride = (uint64_t)E * L.ff;
+    dn.g_off = e->b_off; dn.g_act = small ? e->b_act : nullptr; dn.w_gstride = (uint64_t)E * L.ff;
     if ((r = gemm(e, dn, L.NE, T, false, T * L.top))) return r;
     if (!L.has_shared) return 0;
     if (e->branch_streams) { e->cur = e->side; CK(cudaStreamWaitEvent(e->side, e->ev_fork, 0)); }
@@ -1575,16 +1584,17 @@ int ff_moe_relu2(LayeredEngine *e, const Layer &L, uint32_t T) {
     int r;
     RouteArgs ra{e->h2, L.router, e->b_idx, e->b_wt, e->b_cnt, e->b_off, e->b_fill, e->b_slot, e->b_rows, T, L.NE, L.top, E, L.route_mode};
     ra.groups = L.groups; ra.keep = L.keep_groups; ra.wscale = L.route_scale;
-    if (T <= kGemvMaxM) { if ((r = launch<RouteArgs>(e, k_route_small, dim3(1), dim3(1024), route_smem(L.NE, 1024), ra))) return r; }
+    const bool small = T <= kGemvMaxM;
+    if (small) { ra.act = e->b_act; if ((r = route_small(e, ra))) return r; }
     else if ((r = launch<RouteArgs>(e, k_route, dim3(T), dim3(256), route_smem(L.NE, 256), ra)) ||
              (r = launch<RouteArgs>(e, k_route_place, dim3(1), dim3(1024), 0, ra))) return r;
     GemmArgs u{};
     u.A = e->h2; u.lda = E; u.W = L.up.p; u.ldw = E; u.C = e->b_hb; u.ldc = L.ff; u.M = T; u.N = L.ff; u.K = E; u.a_gmod = 1;
-    u.g_off = e->b_off; u.a_rows = e->b_rows; u.w_gstride = (uint64_t)L.ff * E; u.epi = EPI_RELU2;
+    u.g_off = e->b_off; u.a_rows = e->b_rows; u.g_act = small ? e->b_act : nullptr; u.w_gstride = (uint64_t)L.ff * E; u.epi = EPI_RELU2;
     if ((r = gemm(e, u, L.NE, T, false, T * L.top))) return r;
     GemmArgs dn{};
     dn.A = e->b_hb; dn.lda = L.ff; dn.W = L.down.p; dn.ldw = L.ff; dn.C = e->b_eo; dn.ldc = E; dn.M = T; dn.N = E; dn.K = L.ff; dn.a_gmod = 1;
-    dn.g_off = e->b_off; dn.w_gstride = (uint64_t)E * L.ff;
+    dn.g_off = e->b_off; dn.g_act = small ? e->b_act : nullptr; dn.w_gstride = (uint64_t)E * L.ff;
     return gemm(e, dn, L.NE, T, false, T * L.top);
 }
 
@@ -2520,7 +2530,7 @@ int create(LayeredEngine *e, const nb::ModelDir *dir, uint32_t max_tokens) {
     }
     if (mNE) {
         DM(e->b_idx, T * mTop * 4); DM(e->b_wt, T * mTop * 4); DM(e->b_slot, T * mTop * 4); DM(e->b_rows, T * mTop * 4);
-        DM(e->b_cnt, (size_t)mNE * 4); DM(e->b_off, ((size_t)mNE + 1) * 4); DM(e->b_fill, (size_t)mNE * 4);
+        DM(e->b_cnt, (size_t)mNE * 4); DM(e->b_off, ((size_t)mNE + 1) * 4); DM(e->b_fill, (size_t)mNE * 4); DM(e->b_act, (size_t)kGemvMaxM * mTop * 4);
         CK(cudaMemset(e->b_cnt, 0, (size_t)mNE * 4));
         DM(e->b_hb, T * mFF * 4); DM(e->b_eo, T * mTop * E * 4);
         if (mSFF) { DM(e->b_sh, T * std::max(mSFF, mSFF2) * 4); DM(e->b_so, T * E * 4); }

@@ -49,6 +49,7 @@ enum Epi : uint32_t { EPI_NONE = 0, EPI_BIAS = 1, EPI_GELU_SPLIT = 2, EPI_SIGMOI
 struct GemmArgs {
     const float *A; const void *W; float *C; const float *bias;
     const uint32_t *g_off; const uint32_t *a_rows;
+    const uint32_t *g_act;    // k_gemv with g_off: blockIdx.y is a place in this list of the groups that have rows (0xffffffff past its end)
     uint32_t M, N, K, lda, ldw, ldc;
     uint32_t a_gmod, a_gcols, c_gcols, b_gstride;
     uint64_t w_gstride;
@@ -431,7 +432,9 @@ __device__ __forceinline__ void warp_dots(const WT *wr, const float *(&ap)[kGemv
 // norm in equal parts, EXT 5: the plain product with the residual epilogue, which EXT 4 knows too (registers the plain one keeps)
 template <typename WT, int EXT = 0>
 __device__ __forceinline__ void gemv_body(const GemmArgs &a, float *red) {
-    const GroupView gv = group_view(a, blockIdx.y);
+    const uint32_t group = a.g_act ? a.g_act[blockIdx.y] : blockIdx.y;
+    if (group == 0xffffffffu) return;
+    const GroupView gv = group_view(a, group);
     if (gv.rows == 0) return;
     const uint32_t rows = gv.rows < kGemvMaxM ? gv.rows : kGemvMaxM;
     const uint32_t lane = threadIdx.x & 31u;
@@ -1049,8 +1052,8 @@ __global__ void __launch_bounds__(kAttnWarps * 32, attn_two_blocks(RCH, QT, EXAC
 // in the choice (a gate of a shared expert, computed with the router's precision).  wrow (optional): the weights once more in
 // expert-sorted row order, wrow[slot[t][j]] = wt[t][j], for a product that scales its rows.
 struct RouteArgs { const float *h; const float *router; uint32_t *idx; float *wt; uint32_t *counts; uint32_t *off; uint32_t *fill; uint32_t *slot; uint32_t *rows; uint32_t T, NE, top, E;
-                   uint32_t mode, extra; float *extra_out; float *wrow; uint32_t groups, keep; float wscale; };
-// dynamic shared memory of k_route / k_route_small launched with `threads` threads (NE: rows of the router matrix, extra ones included)
+                   uint32_t mode, extra; float *extra_out; float *wrow; uint32_t groups, keep; float wscale; uint32_t *act; };
+// dynamic shared memory of k_route launched with `threads` threads (NE: rows of the router matrix, extra ones included)
 inline size_t route_smem(uint32_t NE, uint32_t threads) { const uint32_t nw = threads / 32u; return ((size_t)NE + (size_t)NE * (nw > NE ? nw / NE : 1u)) * 4; }
 // router logits of token t into z[NE].  The blockDim/32 warps are dealt out as `ns` slices per expert (ns = warps / NE, at least 1):
 // a warp sums its slice of the row, the slices are added in order.  zp: NE * ns floats of scratch.
@@ -1160,24 +1163,90 @@ __global__ void __launch_bounds__(256) k_route(const RouteArgs a) {
     if (threadIdx.x) return;
     for (uint32_t j = 0; j < a.top; j++) atomicAdd(a.counts + a.idx[(size_t)blockIdx.x * a.top + j], 1u);
 }
-// Short portions: routing and placement of all T tokens in one block of 1024 threads (the one block has the router matrix to itself,
-// so every warp fetches).  Same outputs as k_route + k_route_place; the global counters are not touched.
-__global__ void __launch_bounds__(1024) k_route_small(const RouteArgs a) {
-    pdl_enter();
-    extern __shared__ float z[];
-    uint32_t *cur = reinterpret_cast<uint32_t *>(z);          // after the last token z is free
-    for (uint32_t t = 0; t < a.T; t++) {
-        route_logits(a, t, z, z + a.NE + a.extra);
-        __syncthreads();
-        if (threadIdx.x < 32u) route_pick(a, t, z, z + a.NE + a.extra);
-        __syncthreads();
+// Short portions: routing and placement of all T <= kGemvMaxM tokens in one launch.  A cluster of blocks shares the router's rows (a warp
+// sums a slice of a row for all tokens at once) and hands the logits to its first block, where a warp per token chooses.  Same outputs as
+// k_route + k_route_place; the global counters are not touched.  act (optional): the experts that have rows, 0xffffffff up to T top places.
+constexpr uint32_t kRouteBlocks = 8, kRouteThreads = 512;
+inline size_t route_small_smem(uint32_t NL) { return ((size_t)2 * kGemvMaxM * NL + (size_t)kGemvMaxM * (NL > kRouteThreads / 32u ? NL : kRouteThreads / 32u)) * 4; }
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+__device__ __forceinline__ void st_cluster(float *p, uint32_t rank, float v) {      // *p of block `rank` of this cluster
+    uint32_t at = (uint32_t)__cvta_generic_to_shared(p), there;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(there) : "r"(at), "r"(rank));
+    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(there), "f"(v) : "memory");
+}
+__global__ void __launch_bounds__(kRouteThreads) k_route_small(const RouteArgs a) {
+    pdl_launch_next();
+    cluster_arrive();                          // waited for before the first access to another block's shared memory
+    const uint32_t NL = a.NE + a.extra, rank = blockIdx.x, nb = gridDim.x, nloc = (NL - rank + nb - 1u) / nb;      // this block's rows: rank, rank + nb, ...
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, nw = blockDim.x >> 5, ns = nw > nloc ? nw / nloc : 1u;
+    for (uint32_t i = warp; i < nloc; i += nw) prefetch_weight_rows(a.router, 4u, a.E, a.E, NL, rank + i * nb, NL, 1u);
+    pdl_wait();
+    extern __shared__ float z[];               // [kGemvMaxM][NL] logits (complete in block 0), then scratch
+    float *zg = z + kGemvMaxM * NL, *zp = zg + kGemvMaxM * NL;
+    const bool vec = (a.E & 3u) == 0;
+    const uint32_t per = ((a.E + ns - 1u) / ns + 3u) & ~3u;          // slice length, a multiple of 4
+    for (uint32_t job = warp; job < nloc * ns; job += nw) {
+        const uint32_t sl = job % ns, k0 = min(a.E, sl * per), k1 = min(a.E, k0 + per);
+        const float *w = a.router + (size_t)(rank + job / ns * nb) * a.E;
+        float acc[kGemvMaxM];
+#pragma unroll
+        for (uint32_t t = 0; t < kGemvMaxM; t++) acc[t] = 0.0f;
+        if (vec) {
+            for (uint32_t k = k0 + lane * 4u; k < k1; k += 128u) {
+                const float4 wv = __ldg(reinterpret_cast<const float4 *>(w + k));
+#pragma unroll
+                for (uint32_t t = 0; t < kGemvMaxM; t++)
+                    if (t < a.T) { const float4 hv = *reinterpret_cast<const float4 *>(a.h + (size_t)t * a.E + k); acc[t] = fmaf(hv.w, wv.w, fmaf(hv.z, wv.z, fmaf(hv.y, wv.y, fmaf(hv.x, wv.x, acc[t])))); }
+            }
+        } else
+            for (uint32_t k = k0 + lane; k < k1; k += 32u) {
+                const float wv = w[k];
+#pragma unroll
+                for (uint32_t t = 0; t < kGemvMaxM; t++) if (t < a.T) acc[t] = fmaf(a.h[(size_t)t * a.E + k], wv, acc[t]);
+            }
+#pragma unroll
+        for (uint32_t t = 0; t < kGemvMaxM; t++) {
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], o);
+            if (lane == 0) zp[job * kGemvMaxM + t] = acc[t];
+        }
     }
-    if (threadIdx.x) return;
-    const uint32_t n = a.T * a.top;
-    for (uint32_t e = 0; e < a.NE; e++) cur[e] = 0;
-    for (uint32_t i = 0; i < n; i++) cur[a.idx[i]]++;
-    uint32_t s = 0;
-    for (uint32_t e = 0; e < a.NE; e++) { const uint32_t c = cur[e]; a.off[e] = s; cur[e] = s; s += c; }
+    __syncthreads();
+    cluster_wait();                            // every block of the cluster runs
+    for (uint32_t i = tid; i < nloc * a.T; i += blockDim.x) {
+        const uint32_t t = i / nloc, r = i % nloc, e = rank + r * nb;
+        float v = 0.0f;
+        for (uint32_t sl = 0; sl < ns; sl++) v += zp[(r * ns + sl) * kGemvMaxM + t];
+        st_cluster(z + t * NL + e, 0u, a.mode == 3u && e < a.NE ? sigmoidf_(v) : v);
+    }
+    __syncwarp();
+    cluster_arrive();
+    cluster_wait();
+    if (rank) return;
+    if (warp < a.T) route_pick(a, warp, z + warp * NL, zg + warp * NL);
+    __syncthreads();
+    if (warp) return;
+    uint32_t *cur = reinterpret_cast<uint32_t *>(z), n = a.T * a.top;          // the logits have served
+    for (uint32_t e = lane; e < a.NE; e += 32u) cur[e] = 0;
+    __syncwarp();
+    for (uint32_t i = lane; i < n; i += 32u) atomicAdd(cur + a.idx[i], 1u);
+    __syncwarp();
+    uint32_t s = 0, na = 0;
+    for (uint32_t e0 = 0; e0 < a.NE; e0 += 32u) {
+        const uint32_t e = e0 + lane, c = e < a.NE ? cur[e] : 0u;
+        uint32_t run = c;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) { const uint32_t v = __shfl_up_sync(0xffffffffu, run, o); if (lane >= (uint32_t)o) run += v; }
+        if (e < a.NE) { a.off[e] = s + run - c; cur[e] = s + run - c; }
+        const uint32_t has = __ballot_sync(0xffffffffu, c > 0u);
+        if (a.act && c > 0u) a.act[na + __popc(has & ((1u << lane) - 1u))] = e;
+        na += __popc(has);
+        s += __shfl_sync(0xffffffffu, run, 31);
+    }
+    __syncwarp();
+    if (a.act) for (uint32_t i = na + lane; i < n; i += 32u) a.act[i] = 0xffffffffu;
+    if (lane) return;
     a.off[a.NE] = s;
     for (uint32_t i = 0; i < n; i++) { const uint32_t sl = cur[a.idx[i]]++; a.slot[i] = sl; a.rows[sl] = i / a.top; if (a.wrow) a.wrow[sl] = a.wt[i]; }
 }

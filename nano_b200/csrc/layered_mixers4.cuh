@@ -864,13 +864,6 @@ __device__ __forceinline__ void lane8_dots(const WT *w, const float *x, uint32_t
     for (uint32_t t = 0; t < kGemvMaxM; t++) { acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], 4); acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], 2); acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], 1); }
 }
 constexpr uint32_t kDeltaThreads = 512;    // a block's threads at most (8 per value column; more columns: several passes)
-__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
-__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
-__device__ __forceinline__ void st_cluster(float *p, uint32_t rank, float v) {      // *p of block `rank` of this cluster
-    uint32_t at = (uint32_t)__cvta_generic_to_shared(p), there;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(there) : "r"(at), "r"(rank));
-    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(there), "f"(v) : "memory");
-}
 template <typename WT, int DCH>
 __global__ void __launch_bounds__(kDeltaThreads) k_delta_step(const DeltaStepArgs a) {
     pdl_launch_next();

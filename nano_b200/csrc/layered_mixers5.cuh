@@ -5,8 +5,8 @@
 //   matrix memory        per head  m' = max(f + m, i);  S <- e^(f + m - m') S + e^(i - m') k v^T,  n likewise with k alone;
 //                        o = S^T q / (max(|n . q|, e^(-m')) + 1e-6),  i, f the logs of the gates, soft-capped.
 //                        Long portions run kMemChunk tokens side by side: k_memory_gates (gates, their running sums and the running
-//                        maximum), k_memory_states (the state before every chunk), k_memory_out (all outputs of a chunk: a decayed causal
-//                        product inside it and one product with the state before it).  k_memory_step (short portions): everything from the
+//                        maximum), k_memory_writes (what every chunk writes), k_memory_chain (the state before every chunk), k_memory_out
+//                        (all outputs of a chunk: a decayed causal product inside it and one product with the state before it).  k_memory_step (short portions): everything from the
 //                        joint product's rows to the normed and gated output, a cluster of blocks per head.
 #pragma once
 #include "layered_mixers4.cuh"
@@ -124,95 +124,95 @@ __global__ void __launch_bounds__(1024) k_memory_gates(const MemGatesArgs a) {
     if (threadIdx.x == 0) { a.me[(size_t)h * (a.chunks + 1u) + a.chunks] = m_s; a.m[h] = m_s; }
 }
 
-// The state before every chunk, and at the portion's end.  A block keeps 32 value columns x 64 key coordinates of head h = blockIdx.z in
-// registers (2 columns x 4 coordinates per thread) and walks the chunks; the next chunk's rows are in flight meanwhile.  The blocks of the
-// first value tile carry n beside it.  grid = (value tiles, key tiles, H), 256 threads.
-struct MemStatesArgs { const float *p; uint32_t ld, k0, v0; const double *fb, *fc; const float *me; float *S, *n, *Sin, *nin; uint32_t T, H, D, VD, chunks; };
-__global__ void __launch_bounds__(256, 3) k_memory_states(const MemStatesArgs a) {
+// elements at .. at + 3 of a row of n (zeros past its end, and where !ok); vec: 16-byte loads are aligned
+__device__ __forceinline__ float4 row4(const float *src, uint32_t at, uint32_t n, bool vec, bool ok) {
+    float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (!ok) return v;
+    if (vec) { if (at < n) v = *reinterpret_cast<const float4 *>(src + at); return v; }
+    if (at < n) v.x = src[at];
+    if (at + 1u < n) v.y = src[at + 1u];
+    if (at + 2u < n) v.z = src[at + 2u];
+    if (at + 3u < n) v.w = src[at + 3u];
+    return v;
+}
+// What every chunk writes, relative to the running maximum at its end:  U_c = sum_s e^(F_C - F_s + i_s - m') k_s v_s^T,  and likewise for n.
+// A block makes 64 value columns x 64 key coordinates of one chunk and head, 4 x 4 per thread; the blocks of the first value tile make n
+// too.  grid = (value tiles, key tiles, chunks x H), 256 threads.
+struct MemWriteArgs { const float *p; uint32_t ld, k0, v0; const double *fb, *fc; const float *me; float *U, *Un; uint32_t T, H, D, VD, chunks; };
+__global__ void __launch_bounds__(256, 4) k_memory_writes(const MemWriteArgs a) {
     pdl_enter();
-    __shared__ __align__(16) float k_s[kMemChunk][64], v_s[kMemChunk][32];
-    __shared__ float w_s[kMemChunk], keep_s;
-    const uint32_t tid = threadIdx.x, tx = tid & 15u, ty = tid >> 4, h = blockIdx.z, col0 = blockIdx.x * 32u, d0 = blockIdx.y * 64u, D = a.D, VD = a.VD;
-    const bool vec = ((a.ld | a.k0 | a.v0 | D | VD) & 3u) == 0, with_n = blockIdx.x == 0 && tid < 64u;
-    float4 kr[4], vr[2];
-    float wr[2], keep_r = 0.0f;
-    const float *me = a.me + (size_t)h * (a.chunks + 1u);
-    auto load4 = [&](const float *src, uint32_t at, uint32_t n, bool ok) {      // elements at .. at + 3 of a row of n
-        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (!ok) return v;
-        if (vec) { if (at < n) v = *reinterpret_cast<const float4 *>(src + at); return v; }
-        if (at < n) v.x = src[at];
-        if (at + 1u < n) v.y = src[at + 1u];
-        if (at + 2u < n) v.z = src[at + 2u];
-        if (at + 3u < n) v.w = src[at + 3u];
-        return v;
-    };
-    auto fetch = [&](uint32_t c) {
-        const double end = a.fc[(size_t)h * a.chunks + c] - (double)me[c + 1u];
-        if (tid == 0) keep_r = (float)exp(end + (double)me[c]);
+    __shared__ __align__(16) float k_s[kMemChunk][64], v_s[kMemChunk][64];
+    __shared__ float w_s[kMemChunk];
+    const uint32_t tid = threadIdx.x, tx = tid & 15u, ty = tid >> 4, c = blockIdx.z / a.H, h = blockIdx.z % a.H, col0 = blockIdx.x * 64u, d0 = blockIdx.y * 64u, D = a.D, VD = a.VD;
+    const bool vec = ((a.ld | a.k0 | a.v0 | D | VD) & 3u) == 0;
+    const double end = a.fc[(size_t)h * a.chunks + c] - (double)a.me[(size_t)h * (a.chunks + 1u) + c + 1u];
 #pragma unroll
-        for (uint32_t j = 0; j < 4; j++) { const uint32_t t = c * kMemChunk + ty + 16u * j; kr[j] = load4(a.p + (size_t)t * a.ld + a.k0 + h * D, d0 + tx * 4u, D, t < a.T); }
-#pragma unroll
-        for (uint32_t j = 0; j < 2; j++) {
-            const uint32_t t = c * kMemChunk + (tid >> 3) + 32u * j;
-            vr[j] = load4(a.p + (size_t)t * a.ld + a.v0 + h * VD, col0 + (tid & 7u) * 4u, VD, t < a.T);
-            wr[j] = t < a.T ? expf((float)(a.fb[(size_t)h * a.T + t] + end)) : 0.0f;
-        }
-    };
-    float S[2][4], nv = 0.0f;
-#pragma unroll
-    for (uint32_t c = 0; c < 2; c++)
-#pragma unroll
-        for (uint32_t e = 0; e < 4; e++) { const uint32_t col = col0 + ty * 2u + c, d = d0 + tx * 4u + e; S[c][e] = (col < VD && d < D) ? a.S[((size_t)h * VD + col) * D + d] : 0.0f; }
-    if (with_n && d0 + tid < D) nv = a.n[(size_t)h * D + d0 + tid];
-    auto put = [&](float *dst, float *ndst) {      // dst [VD][D] and ndst [D] of this head
-#pragma unroll
-        for (uint32_t c = 0; c < 2; c++) {
-            const uint32_t col = col0 + ty * 2u + c, d = d0 + tx * 4u;
-            if (col >= VD) continue;
-            float *q = dst + (size_t)col * D + d;
-            if (vec) { if (d < D) *reinterpret_cast<float4 *>(q) = make_float4(S[c][0], S[c][1], S[c][2], S[c][3]); }
-            else {
-#pragma unroll
-                for (uint32_t e = 0; e < 4; e++) if (d + e < D) q[e] = S[c][e];
-            }
-        }
-        if (with_n && d0 + tid < D) ndst[d0 + tid] = nv;
-    };
-    fetch(0);
-    for (uint32_t c = 0; c < a.chunks; c++) {
-        __syncthreads();                       // the chunk before has been read
-#pragma unroll
-        for (uint32_t j = 0; j < 4; j++) *reinterpret_cast<float4 *>(&k_s[ty + 16u * j][tx * 4u]) = kr[j];
-#pragma unroll
-        for (uint32_t j = 0; j < 2; j++) {
-            const uint32_t s = (tid >> 3) + 32u * j;
-            *reinterpret_cast<float4 *>(&v_s[s][(tid & 7u) * 4u]) = make_float4(vr[j].x * wr[j], vr[j].y * wr[j], vr[j].z * wr[j], vr[j].w * wr[j]);
-            if ((tid & 7u) == 0) w_s[s] = wr[j];
-        }
-        if (tid == 0) keep_s = keep_r;
-        __syncthreads();
-        if (c + 1u < a.chunks) fetch(c + 1u);
-        put(a.Sin + ((size_t)c * a.H + h) * VD * D, a.nin + ((size_t)c * a.H + h) * D);
-        const float keep = keep_s;
-#pragma unroll
-        for (uint32_t j = 0; j < 2; j++)
-#pragma unroll
-            for (uint32_t e = 0; e < 4; e++) S[j][e] *= keep;
-        nv *= keep;
+    for (uint32_t j = 0; j < 4; j++) {
+        const uint32_t s = ty + 16u * j, t = c * kMemChunk + s;
+        const float *row = a.p + (size_t)t * a.ld;
+        const float w = t < a.T ? expf((float)(a.fb[(size_t)h * a.T + t] + end)) : 0.0f;
+        const float4 k = row4(row + a.k0 + h * D, d0 + tx * 4u, D, vec, t < a.T), v = row4(row + a.v0 + h * VD, col0 + tx * 4u, VD, vec, t < a.T);
+        *reinterpret_cast<float4 *>(&k_s[s][tx * 4u]) = k;
+        *reinterpret_cast<float4 *>(&v_s[s][tx * 4u]) = make_float4(v.x * w, v.y * w, v.z * w, v.w * w);
+        if (tx == 0) w_s[s] = w;
+    }
+    __syncthreads();
+    float u[4][4] = {}, un = 0.0f;             // u[column][coordinate]
 #pragma unroll 8
-        for (uint32_t s = 0; s < kMemChunk; s++) {
-            const float4 k = *reinterpret_cast<const float4 *>(&k_s[s][tx * 4u]);
-            const float2 v = *reinterpret_cast<const float2 *>(&v_s[s][ty * 2u]);
-            S[0][0] = fmaf(k.x, v.x, S[0][0]); S[0][1] = fmaf(k.y, v.x, S[0][1]); S[0][2] = fmaf(k.z, v.x, S[0][2]); S[0][3] = fmaf(k.w, v.x, S[0][3]);
-            S[1][0] = fmaf(k.x, v.y, S[1][0]); S[1][1] = fmaf(k.y, v.y, S[1][1]); S[1][2] = fmaf(k.z, v.y, S[1][2]); S[1][3] = fmaf(k.w, v.y, S[1][3]);
-        }
-        if (with_n) {
-#pragma unroll 8
-            for (uint32_t s = 0; s < kMemChunk; s++) nv = fmaf(w_s[s], k_s[s][tid], nv);
+    for (uint32_t s = 0; s < kMemChunk; s++) {
+        const float4 k = *reinterpret_cast<const float4 *>(&k_s[s][tx * 4u]), v = *reinterpret_cast<const float4 *>(&v_s[s][ty * 4u]);
+        const float kk[4] = {k.x, k.y, k.z, k.w}, vv[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (uint32_t i = 0; i < 4; i++)
+#pragma unroll
+            for (uint32_t j = 0; j < 4; j++) u[i][j] = fmaf(vv[i], kk[j], u[i][j]);
+    }
+    float *dst = a.U + ((size_t)c * a.H + h) * VD * D;
+#pragma unroll
+    for (uint32_t i = 0; i < 4; i++) {
+        const uint32_t col = col0 + ty * 4u + i, d = d0 + tx * 4u;
+        if (col >= VD) continue;
+        float *q = dst + (size_t)col * D + d;
+        if (vec) { if (d < D) *reinterpret_cast<float4 *>(q) = make_float4(u[i][0], u[i][1], u[i][2], u[i][3]); }
+        else {
+#pragma unroll
+            for (uint32_t e = 0; e < 4; e++) if (d + e < D) q[e] = u[i][e];
         }
     }
-    put(a.S + (size_t)h * VD * D, a.n + (size_t)h * D);
+    if (blockIdx.x == 0 && tid < 64u && d0 + tid < D) {
+#pragma unroll 8
+        for (uint32_t s = 0; s < kMemChunk; s++) un = fmaf(w_s[s], k_s[s][tid], un);
+        a.Un[((size_t)c * a.H + h) * D + d0 + tid] = un;
+    }
+}
+
+// In place: U_c becomes the state before chunk c (S, n: the state before the portion, afterwards the one behind it).  A thread walks one
+// coordinate of the state (or of n) through the chunks, eight loads in flight.  grid = (blocks over VD D + D, H), 256 threads.
+struct MemChainArgs { const double *fc; const float *me; float *S, *n, *U, *Un; uint32_t H, D, VD, chunks; };
+__global__ void __launch_bounds__(256) k_memory_chain(const MemChainArgs a) {
+    pdl_enter();
+    __shared__ float keep_s[256];
+    const uint32_t h = blockIdx.y, tid = threadIdx.x, i = blockIdx.x * 256u + tid, nS = a.VD * a.D, total = nS + a.D;
+    const bool live = i < total, isS = i < nS;
+    float *st = isS ? a.S + (size_t)h * nS + i : a.n + (size_t)h * a.D + (i - nS), *u = isS ? a.U + (size_t)h * nS + i : a.Un + (size_t)h * a.D + (i - nS);
+    const size_t step = (size_t)a.H * (isS ? nS : a.D);
+    float s = live ? *st : 0.0f;
+    for (uint32_t base = 0; base < a.chunks; base += 256u) {
+        const uint32_t n = min(256u, a.chunks - base);
+        __syncthreads();
+        if (tid < n) { const float *me = a.me + (size_t)h * (a.chunks + 1u) + base + tid; keep_s[tid] = (float)exp(a.fc[(size_t)h * a.chunks + base + tid] + (double)me[0] - (double)me[1]); }
+        __syncthreads();
+        if (!live) continue;
+        for (uint32_t c0 = 0; c0 < n; c0 += 8u) {
+            float v[8];
+#pragma unroll
+            for (uint32_t k = 0; k < 8; k++) v[k] = c0 + k < n ? u[(base + c0 + k) * step] : 0.0f;
+#pragma unroll
+            for (uint32_t k = 0; k < 8; k++)
+                if (c0 + k < n) { u[(base + c0 + k) * step] = s; s = fmaf(keep_s[c0 + k], s, v[k]); }
+        }
+    }
+    if (live) *st = s;
 }
 
 // All outputs of chunk c = blockIdx.y of head h = blockIdx.z for 64 VJ value columns.  A thread owns 4 tokens x 4 VJ columns.  The key
@@ -234,16 +234,6 @@ __global__ void __launch_bounds__(256, 2) k_memory_out(const MemOutArgs a) {
     const uint32_t tid = threadIdx.x, tx = tid & 15u, ty = tid >> 4, h = blockIdx.z, c = blockIdx.y, col0 = blockIdx.x * VT, D = a.D, VD = a.VD, t0 = c * kMemChunk;
     const bool vec = ((a.ld | a.q0 | a.k0 | a.v0 | D | VD) & 3u) == 0;
     const float *Sin = a.Sin + ((size_t)c * a.H + h) * VD * D, *nin = a.nin + ((size_t)c * a.H + h) * D;
-    auto load4 = [&](const float *src, uint32_t at, uint32_t n, bool ok) {      // elements at .. at + 3 of a row of n
-        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (!ok) return v;
-        if (vec) { if (at < n) v = *reinterpret_cast<const float4 *>(src + at); return v; }
-        if (at < n) v.x = src[at];
-        if (at + 1u < n) v.y = src[at + 1u];
-        if (at + 2u < n) v.z = src[at + 2u];
-        if (at + 3u < n) v.w = src[at + 3u];
-        return v;
-    };
     float s[4][4] = {}, o[4][VJ * 4] = {}, nq[4] = {};
     float4 qr[2], kr[2], Sr[VJ * 2]; float nr = 0.0f;
     auto fetch = [&](uint32_t d0) {
@@ -252,10 +242,10 @@ __global__ void __launch_bounds__(256, 2) k_memory_out(const MemOutArgs a) {
         for (uint32_t j = 0; j < 2; j++) {
             const uint32_t t = t0 + (tid >> 3) + 32u * j;
             const float *row = a.p + (size_t)t * a.ld + h * D;
-            qr[j] = load4(row + a.q0, e, D, t < a.T); kr[j] = load4(row + a.k0, e, D, t < a.T);
+            qr[j] = row4(row + a.q0, e, D, vec, t < a.T); kr[j] = row4(row + a.k0, e, D, vec, t < a.T);
         }
 #pragma unroll
-        for (uint32_t j = 0; j < VJ * 2u; j++) { const uint32_t col = col0 + (tid >> 3) + 32u * j; Sr[j] = load4(Sin + (size_t)col * D, e, D, col < VD); }
+        for (uint32_t j = 0; j < VJ * 2u; j++) { const uint32_t col = col0 + (tid >> 3) + 32u * j; Sr[j] = row4(Sin + (size_t)col * D, e, D, vec, col < VD); }
         if (tid < kMemSlice) nr = d0 + tid < D ? nin[d0 + tid] : 0.0f;
     };
     fetch(0);
@@ -303,7 +293,7 @@ __global__ void __launch_bounds__(256, 2) k_memory_out(const MemOutArgs a) {
     __syncthreads();                           // the slices have been read: the weights and the values take their place
     for (uint32_t i = tid; i < kMemChunk * (VT / 4u); i += 256u) {
         const uint32_t k = i / (VT / 4u), e = (i % (VT / 4u)) * 4u;
-        *reinterpret_cast<float4 *>(v_s + k * VT + e) = load4(a.p + (size_t)(t0 + k) * a.ld + a.v0 + h * VD, col0 + e, VD, t0 + k < a.T);
+        *reinterpret_cast<float4 *>(v_s + k * VT + e) = row4(a.p + (size_t)(t0 + k) * a.ld + a.v0 + h * VD, col0 + e, VD, vec, t0 + k < a.T);
     }
     const double *fa = a.fa + (size_t)h * a.T, *fb = a.fb + (size_t)h * a.T;
     const float *mt = a.mt + (size_t)h * a.T;
