@@ -1422,8 +1422,8 @@ int mix_memory(LayeredEngine *e, const Layer &L, const Run &run, const Ctx &cx) 
     if ((r = launch<MemGatesArgs>(e, k_memory_gates, dim3(H), dim3(1024), 0, ga)) ||
         (r = launch<MemWriteArgs>(e, k_memory_writes, dim3((VD + 63u) / 64u, (D + 63u) / 64u, chunks * H), dim3(256), 0, wa)) ||
         (r = launch<MemChainArgs>(e, k_memory_chain, dim3((VD * D + D + 255u) / 256u, H), dim3(256), 0, ca))) return r;
-    // 128 value columns per block (the scores are made once for them) where that still fills the GPU twice
-    if (VD > 64u && (VD + 127u) / 128u * chunks * H >= 2u * (uint32_t)e->num_sms) r = launch<MemOutArgs>(e, k_memory_out<2>, dim3((VD + 127u) / 128u, chunks, H), dim3(256), memory_out_smem(2), oa);
+    // 128 value columns per block (the scores are made once for them) where that still gives every SM a block
+    if (VD > 64u && (VD + 127u) / 128u * chunks * H >= (uint32_t)e->num_sms) r = launch<MemOutArgs>(e, k_memory_out<2>, dim3((VD + 127u) / 128u, chunks, H), dim3(256), memory_out_smem(2), oa);
     else r = launch<MemOutArgs>(e, k_memory_out<1>, dim3((VD + 63u) / 64u, chunks, H), dim3(256), memory_out_smem(1), oa);
     if (r) return r;
     RetOutArgs na{e->b_mo, e->b_p + g0, P, e->b_a, T, H, VD, e->eps, L.gn, 1u, VD};
@@ -1601,11 +1601,16 @@ int ff_moe_relu2(LayeredEngine *e, const Layer &L, uint32_t T) {
 // x = rms_norm(alpha x + sublayer output) w; moe: the output is the chosen experts' rows, else e->d
 int post_ln(LayeredEngine *e, const Layer *moe, const float *w, float *keep, uint32_t T) {
     PostLnArgs a{e->x, e->d, moe ? e->b_eo : nullptr, e->b_slot, e->b_wt, moe ? moe->top : 0u, w, e->alpha, keep, T, e->E, e->eps};
+    const uint32_t vw = e->E % 4u ? 1u : 4u, runs = e->E / vw;
     // a short portion is a few lone blocks: wide ones, so that a thread's chain of loads stays short
-    const uint32_t per = T <= kGemvMaxM ? 2u : 8u, threads = std::min(1024u, std::max(128u, (e->E / per + 31u) & ~31u));
-    if (e->E <= 2u * threads) return launch<PostLnArgs>(e, k_post_ln<2>, dim3(T), dim3(threads), 0, a);
-    if (e->E <= 8u * threads) return launch<PostLnArgs>(e, k_post_ln<8>, dim3(T), dim3(threads), 0, a);
-    return launch<PostLnArgs>(e, k_post_ln<0>, dim3(T), dim3(threads), 0, a);
+    const uint32_t per = T <= kGemvMaxM ? 1u : 2u, threads = std::min(1024u, std::max(64u, (runs / per + 31u) & ~31u)), nv = (runs + threads - 1u) / threads;
+    if (vw == 4u) {
+        if (nv <= 1u) return launch<PostLnArgs>(e, k_post_ln<1, 4>, dim3(T), dim3(threads), 0, a);
+        if (nv <= 2u) return launch<PostLnArgs>(e, k_post_ln<2, 4>, dim3(T), dim3(threads), 0, a);
+        return launch<PostLnArgs>(e, k_post_ln<0, 4>, dim3(T), dim3(threads), 0, a);
+    }
+    if (nv <= 2u) return launch<PostLnArgs>(e, k_post_ln<2, 1>, dim3(T), dim3(threads), 0, a);
+    return launch<PostLnArgs>(e, k_post_ln<0, 1>, dim3(T), dim3(threads), 0, a);
 }
 
 // every layer run over T tokens (x already holds their embeddings) of the sequence in `slot`, whose first token sits at pos0

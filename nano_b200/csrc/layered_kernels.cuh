@@ -1254,10 +1254,18 @@ __global__ void __launch_bounds__(kRouteThreads) k_route_small(const RouteArgs a
 // (token t, choice j) in the expert-sorted order and rows[slot] = t
 __global__ void __launch_bounds__(1024) k_route_place(const RouteArgs a) {
     pdl_enter();
-    if (threadIdx.x == 0) {
+    if (threadIdx.x < 32u) {
+        const uint32_t lane = threadIdx.x;
         uint32_t s = 0;
-        for (uint32_t e = 0; e < a.NE; e++) { a.off[e] = s; s += a.counts[e]; a.counts[e] = 0; a.fill[e] = 0; }
-        a.off[a.NE] = s;
+        for (uint32_t e0 = 0; e0 < a.NE; e0 += 32u) {
+            const uint32_t e = e0 + lane, c = e < a.NE ? a.counts[e] : 0u;
+            uint32_t run = c;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) { const uint32_t v = __shfl_up_sync(0xffffffffu, run, o); if (lane >= (uint32_t)o) run += v; }
+            if (e < a.NE) { a.off[e] = s + run - c; a.counts[e] = 0; a.fill[e] = 0; }
+            s += __shfl_sync(0xffffffffu, run, 31);
+        }
+        if (lane == 0) a.off[a.NE] = s;
     }
     __syncthreads();
     for (uint32_t i = threadIdx.x; i < a.T * a.top; i += blockDim.x) {

@@ -16,46 +16,72 @@ namespace lm {
 
 // ------------------------------------------------------------------------------------------------
 // x[t] = u / rms(u) w  with  u = alpha x[t] + d[t],  or (eo given)  u = alpha x[t] + sum_j wt[t][j] eo[slot[t][j]];  keep (optional)
-// receives the updated x.  One block per token; NV > 0: a thread keeps its (at most NV) elements in registers across the reduction.
+// receives the updated x.  One block per token.  NV > 0: a thread keeps its (at most NV) runs of VW neighbours in registers across the
+// reduction; VW 4: rows are multiples of 4 and travel in 16-byte pieces.
 // ------------------------------------------------------------------------------------------------
 struct PostLnArgs { float *x; const float *d; const float *eo; const uint32_t *slot; const float *wt; uint32_t top; const float *w; float alpha; float *keep; uint32_t T, E; float eps; };
-template <int NV>
+template <int VW> __device__ __forceinline__ void stg_vec(float *p, const float (&v)[VW]) {
+    if constexpr (VW == 4) *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else *p = v[0];
+}
+template <int NV, int VW>
 __global__ void __launch_bounds__(1024) k_post_ln(const PostLnArgs a) {
     pdl_enter();
     __shared__ float red[32];
     const uint32_t t = blockIdx.x;
     const size_t row = (size_t)t * a.E;
     float *x = a.x + row;
-    auto sum_at = [&](uint32_t i) {
-        float y = 0.0f;
-        if (a.eo) { for (uint32_t j = 0; j < a.top; j++) y = fmaf(a.wt[(size_t)t * a.top + j], a.eo[(size_t)a.slot[(size_t)t * a.top + j] * a.E + i], y); }
-        else y = a.d[row + i];
-        return fmaf(a.alpha, x[i], y);
+    auto sum_at = [&](uint32_t i, float (&u)[VW]) {
+        float xv[VW];
+        lds_vec<VW>(x + i, xv);
+        if (a.eo) {
+#pragma unroll
+            for (int e = 0; e < VW; e++) u[e] = 0.0f;
+            for (uint32_t j = 0; j < a.top; j++) {
+                const float wt = a.wt[(size_t)t * a.top + j];
+                float v[VW];
+                lds_vec<VW>(a.eo + (size_t)a.slot[(size_t)t * a.top + j] * a.E + i, v);
+#pragma unroll
+                for (int e = 0; e < VW; e++) u[e] = fmaf(wt, v[e], u[e]);
+            }
+        } else lds_vec<VW>(a.d + row + i, u);
+#pragma unroll
+        for (int e = 0; e < VW; e++) u[e] = fmaf(a.alpha, xv[e], u[e]);
     };
-    float u[NV > 0 ? NV : 1], s = 0.0f;
+    auto store = [&](uint32_t i, const float (&u)[VW], float rinv) {
+        float w[VW];
+        lds_vec<VW>(a.w + i, w);
+#pragma unroll
+        for (int e = 0; e < VW; e++) w[e] *= u[e] * rinv;
+        stg_vec<VW>(x + i, w);
+        if (a.keep) stg_vec<VW>(a.keep + row + i, w);
+    };
+    float u[NV > 0 ? NV : 1][VW], s = 0.0f;
     if constexpr (NV > 0) {
 #pragma unroll
         for (int k = 0; k < NV; k++) {
-            const uint32_t i = threadIdx.x + k * blockDim.x;
-            u[k] = i < a.E ? sum_at(i) : 0.0f;
-            s = fmaf(u[k], u[k], s);
+            const uint32_t i = (threadIdx.x + k * blockDim.x) * VW;
+            if (i < a.E) {
+                sum_at(i, u[k]);
+#pragma unroll
+                for (int e = 0; e < VW; e++) s = fmaf(u[k][e], u[k][e], s);
+            }
         }
     } else {
-        for (uint32_t i = threadIdx.x; i < a.E; i += blockDim.x) { const float v = sum_at(i); x[i] = v; s = fmaf(v, v, s); }      // a thread reads back only what it wrote
+        for (uint32_t i = threadIdx.x * VW; i < a.E; i += blockDim.x * VW) {      // a thread reads back only what it wrote
+            sum_at(i, u[0]);
+            stg_vec<VW>(x + i, u[0]);
+#pragma unroll
+            for (int e = 0; e < VW; e++) s = fmaf(u[0][e], u[0][e], s);
+        }
     }
     s = block_sum(s, red);
     const float rinv = 1.0f / sqrtf(s / (float)a.E + a.eps);
     if constexpr (NV > 0) {
 #pragma unroll
-        for (int k = 0; k < NV; k++) {
-            const uint32_t i = threadIdx.x + k * blockDim.x;
-            if (i >= a.E) continue;
-            const float v = u[k] * rinv * a.w[i];
-            x[i] = v;
-            if (a.keep) a.keep[row + i] = v;
-        }
+        for (int k = 0; k < NV; k++) { const uint32_t i = (threadIdx.x + k * blockDim.x) * VW; if (i < a.E) store(i, u[k], rinv); }
     } else
-        for (uint32_t i = threadIdx.x; i < a.E; i += blockDim.x) { const float v = x[i] * rinv * a.w[i]; x[i] = v; if (a.keep) a.keep[row + i] = v; }
+        for (uint32_t i = threadIdx.x * VW; i < a.E; i += blockDim.x * VW) { lds_vec<VW>(x + i, u[0]); store(i, u[0], rinv); }
 }
 
 // ------------------------------------------------------------------------------------------------

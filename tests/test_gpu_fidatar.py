@@ -182,15 +182,16 @@ def test_ragged_widths(tmp_path, width, vocab):
     eng.close()
 
 
-def test_very_wide_residual(tmp_path):
-    """a residual wider than the registers of the norm's block hold"""
-    check_alone(tmp_path, md.fidatar_config(16, 8400, [("mlstm", mem(heads=1, dim=8, vdim=8), dense(16))]), n=9)
+@pytest.mark.parametrize("width", [2051, 4100, 8400])
+def test_wide_residual(tmp_path, width):
+    """residuals wider than the registers of the norm's block hold, with and without 16-byte rows"""
+    check_alone(tmp_path, md.fidatar_config(16, width, [("mlstm", mem(heads=1, dim=8, vdim=8), dense(16))]), n=9)
 
 
 def mixed_cfg(vocab=67):
     layers = [("attention", att(), dense(40)), ("mlstm", MEM, MOE), ("attention", att(heads=3, kv_heads=3, dim=8, mask={"size": 64}, rot={"dims": 4, "base": 40.0}), None),
               ("mlstm", mem(heads=2, dim=36, gate_cap=14.0), dense(24)), ("attention", att(mask={"size": 30}), moe(8, 2, 4, 3))]
-    return md.fidatar_config(vocab, 56, layers)
+    return md.fidatar_config(vocab, 56, layers, alpha=2.5)          # a calm residual: five layers of this size amplify a rounding some fifty times at 1.5
 
 
 @pytest.mark.parametrize("order", ["m", "a", "am", "mam", "aamm", "AmMa", "MAXY"])
