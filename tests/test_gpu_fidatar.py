@@ -533,7 +533,7 @@ def test_model_constants(tmp_path, kw):
 
 def test_long_prompt_splits_keys_in_decoding(tmp_path):
     """Short portions deal the key pages out to several blocks and merge; past 64 pages a block takes several of them; prompts longer than
-    one portion of the engine's own; many chunks of the memory, more than one round of its gates."""
+    one portion of the engine's own; many chunks of the memory, more than one pass of its gates kernel."""
     cfg = md.fidatar_config(40, 48, [("attention", att(heads=3, kv_heads=1, mask=None), dense(24)), ("mlstm", MEM, None), ("attention", att(heads=3, kv_heads=1, mask={"size": 1500}), None)])
     eng, w = build(tmp_path, cfg, max_tokens=400)
     t = toks(cfg, 330, seed=6)
